@@ -74,13 +74,19 @@ class PageTableHost:
 
     `window` > 0 means that only the last `window` positions of a sequence are ever read, so
     pages wholly below that range are given back after each step (`trim`); with `keep_first` > 0 the
-    first that many positions are read for ever as well, and the pages that hold them stay."""
+    first that many positions are read for ever as well, and the pages that hold them stay. `chunk` > 0 means that a
+    position reads only its own chunk of that many positions (chunks counted from position 0): pages wholly below the
+    next position's chunk are given back."""
 
-    def __init__(self, n_pages: int, page_size: int, max_pages_per_seq: int, window: int = 0, keep_first: int = 0):
+    def __init__(self, n_pages: int, page_size: int, max_pages_per_seq: int, window: int = 0, keep_first: int = 0,
+                 chunk: int = 0):
+        if window > 0 and chunk > 0:
+            raise ValueError("a group has a window or chunks, not both")
         self.pages = FreeList(n_pages, "page")
         self.page_size = page_size
         self.max_pages_per_seq = max_pages_per_seq
         self.window = window
+        self.chunk = chunk
         self.keep_first = max(0, keep_first) if window > 0 else 0
         self._held: Dict[int, Dict[int, int]] = {}      # slot -> {logical page: physical page}
 
@@ -112,11 +118,12 @@ class PageTableHost:
         return list(zip(missing, phys))
 
     def trim(self, slot: int, length: int) -> List[int]:
-        """Gives back pages that no later token of this slot can read (window groups only)."""
-        if self.window <= 0:
+        """Gives back pages that no later token of this slot can read (groups with a window or chunks only)."""
+        if self.window <= 0 and self.chunk <= 0:
             return []
         held = self._held[slot]
-        first = max(0, length + 1 - self.window) // self.page_size
+        lowest = length // self.chunk * self.chunk if self.chunk > 0 else max(0, length + 1 - self.window)
+        first = lowest // self.page_size
         kept = (self.keep_first + self.page_size - 1) // self.page_size      # pages of the positions kept for ever
         dead = [lp for lp in held if kept <= lp < first]
         for lp in dead:

@@ -2,14 +2,14 @@
 
 Layout. A *unit* is the storage of one entry of the model's run order (a layer that runs
 twice has two units; a layer that reads another entry's cache has none). Units whose mixers
-ask for the same thing (KV heads, head sizes, window, kept first positions) form a *group* with storage of its own:
+ask for the same thing (KV heads, head sizes, window or chunk, kept first positions) form a *group* with storage of its own:
 
     k, v          [units, pages + 1, kv_heads, page_size, head_dim]   keys are stored rotated
     block_table   [slots + 1, max_pages_per_seq] int32                logical page -> page
 
 Pages hold `page_size` (64) consecutive positions of one sequence; a sequence holds only the
 pages it has reached, so memory follows the tokens held, not slots x longest length. A group
-with a window gives pages back once no later token can read them (the pages of the first
+with a window or chunks gives pages back once no later token can read them (the pages of the first
 `keep_first` positions, where a request names some, are never among them). Fixed-size per-sequence state
 (for mixers that carry a recurrent state) lives beside it as [units, slots + 1, *shape] and is
 zeroed when a slot is taken; this architecture asks for none. A unit may hold several requests of
@@ -45,6 +45,8 @@ class KVRequest:
     name: str = "kv"
     v_head_dim: Optional[int] = None
     keep_first: int = 0
+    # n > 0: a position reads only its own chunk of n positions, counted from position 0 (excludes a window)
+    chunk: int = 0
     # n > 0: the values ARE the first n columns of the key rows (a latent that serves as key and value at once);
     # no value storage is made, `v` is a view into `k`, and v_head_dim is n
     values_in_keys: int = 0
@@ -61,8 +63,8 @@ class KVRequest:
         return self.n_kv_heads * (self.head_dim + (0 if self.values_in_keys else self.value_dim))
 
     def geometry(self) -> Tuple[int, int, int, int, int, int]:
-        """What decides which group's storage serves the request."""
-        return (self.n_kv_heads, self.head_dim, self.window, self.value_dim, self.keep_first if self.window else 0,
+        """What decides which group's storage serves the request (a chunk stands as a negative window)."""
+        return (self.n_kv_heads, self.head_dim, -self.chunk if self.chunk else self.window, self.value_dim, self.keep_first if self.window else 0,
                 self.values_in_keys)
 
 
@@ -108,7 +110,7 @@ class _KVGroup:
                  dtype: torch.dtype, device):
         self.req = req
         self.units = units
-        self.table = PageTableHost(n_pages, PAGE_SIZE, max_pages_per_seq, req.window, req.keep_first)
+        self.table = PageTableHost(n_pages, PAGE_SIZE, max_pages_per_seq, req.window, req.keep_first, req.chunk)
         shape = (len(units), n_pages + 1, req.n_kv_heads, PAGE_SIZE)
         self.k = torch.zeros(shape + (req.head_dim,), dtype=dtype, device=device)
         if req.values_in_keys:

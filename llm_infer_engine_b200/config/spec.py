@@ -81,9 +81,11 @@ class LayerSpec:
 class LayerCall:
     """One entry of the run order. `layer` indexes `ModelSpec.layers`; a layer may appear in
     several entries. Each entry owns a cache unit of its own unless `cache_of` names an
-    EARLIER entry of the schedule, whose unit it then reads instead of writing one."""
+    EARLIER entry of the schedule, whose unit it then reads instead of writing one. `before` names
+    a stage of `ModelSpec.stages` that runs on the residual stream right before this entry."""
     layer: int
     cache_of: Optional[int] = None
+    before: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -108,12 +110,17 @@ class ModelSpec:
     after_head: Optional[PartSpec] = None
     after_embedding_name: str = "after_embedding"
     after_head_name: str = "after_head"
+    # Stages between layers (group "stream") by name; an entry of the schedule names the one that runs before it. A
+    # stage's tensors live under its name.
+    stages: Mapping[str, PartSpec] = field(default_factory=dict)
 
     def validate(self) -> None:
         n = len(self.layers)
         for pos, call in enumerate(self.schedule):
             if not 0 <= call.layer < n:
                 raise ValueError(f"schedule[{pos}] names layer {call.layer}, but there are {n} layers")
+            if call.before is not None and call.before not in self.stages:
+                raise ValueError(f"schedule[{pos}].before names the stage {call.before!r}, which there is none of")
             if call.cache_of is not None:
                 if not 0 <= call.cache_of < pos:
                     raise ValueError(

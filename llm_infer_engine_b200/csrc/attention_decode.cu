@@ -38,7 +38,7 @@ __device__ __forceinline__ void load_vec<float, 4>(const float* p, float (&out)[
 
 // The visible key range of a sequence that holds `len` tokens after this step: [lo, len).
 __device__ __forceinline__ int first_visible(int len, int window) {
-  return (window > 0 && len - window > 0) ? len - window : 0;
+  return first_visible_key(max(len - 1, 0), window);
 }
 
 // One block = one cache page (64 keys) of one KV head of one sequence, for all its query heads. A

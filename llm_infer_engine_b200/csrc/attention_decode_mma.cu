@@ -27,9 +27,8 @@ namespace llmie {
 
 constexpr int kMdPage = 64;
 
-__device__ __forceinline__ int md_first_visible(int len, int window) {
-  return (window > 0 && len - window > 0) ? len - window : 0;
-}
+// the newest token's view (len >= 1: its position is len - 1)
+__device__ __forceinline__ int md_first_visible(int len, int window) { return first_visible_key(max(len - 1, 0), window); }
 __device__ __forceinline__ void md_mma(float (&c)[4], unsigned a0, unsigned a1, unsigned a2, unsigned a3, unsigned b0,
                                        unsigned b1) {
   asm volatile(

@@ -65,6 +65,7 @@ struct AttnShared {
   uint64_t p_ready, pv_full;
   uint32_t tmem_base;
   int abort;
+  int last_lo;                     // the first key the tile's last query row may see: the latest among its rows
   // the two threads of a query row tell each other their maxima (and, at the end, their sums) through
   // shared memory; the two warps that share a quarter of the rows meet at an mbarrier of their own
   // (a bounded wait that sleeps in hardware, so a waiting warp does not take issue slots from its partner
@@ -161,7 +162,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   const int rows_here = min(kQTile, q_len - t0);
   // keys this tile of queries may see: [first_key, last_key]
   const int last_key = start + t0 + rows_here - 1;
-  const int first_key = (window > 0 && start + t0 - window + 1 > 0) ? start + t0 - window + 1 : 0;
+  const int first_key = first_visible_key(start + t0, window);
   const int tile_lo = first_key / kKTile, tile_hi = last_key / kKTile;
   // With kept first keys (keys below keep_first stay visible behind the window) the key tiles that hold them come
   // first, as far as they lie below the window's tiles; then the window's tiles. tile_of(jt) is the key tile of step jt.
@@ -214,6 +215,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     mbar_init(&sh.pv_full, 1);
     for (int i = 0; i < 4; ++i) mbar_init(&sh.pair_bar[i], 64);
     sh.abort = 0;
+    sh.last_lo = first_visible_key(start + t0 + kQTile - 1, window);
     fence_mbar_init();
     // The first loads leave at once, while warp 1 still asks for tensor memory: only this thread touches the
     // barriers they complete on until the block has met below.
@@ -321,7 +323,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const int r = quarter * 32 + lane;                   // row of the tile = TMEM lane
     const uint32_t lane_addr = tmem + ((uint32_t)(quarter * 32) << 16);
     const int qpos = start + t0 + r;                     // absolute position of this query
-    const int lo = (window > 0 && qpos - window + 1 > 0) ? qpos - window + 1 : 0;
+    const int lo = first_visible_key(qpos, window);
     const float sl2 = scale * 1.4426950408889634f;       // exp(x * scale) = exp2(x * scale * log2 e)
     const float sig_b = SIGMOID ? so.sigmoid_bias[head] * 1.4426950408889634f : 0.f;
     constexpr int kCols = kKTile / 2;                    // key columns of a tile this thread handles
@@ -371,7 +373,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       const int tile = tile_of(jt);
       const int kbase = tile * kKTile + half * kCols;
       const bool edge = (tile * kKTile + kKTile - 1 > start + t0) ||
-                        (window > 0 && tile * kKTile < start + t0 + kQTile - window);
+                        tile * kKTile < sh.last_lo;
       // pass 1: the row's maximum over the keys it may see
       // (four running maxima and, below, four running sums: one chain of 64 dependent operations would be
       // what a row's time consists of)
@@ -583,7 +585,8 @@ extern "C" int llmie_attention_prefill_tc_supported(int hd, int page_size) {
 // caches: bfloat16 [n_pages_total, n_kv, 64, hd]; the LAST page (n_pages_total - 1) is a scratch
 // page that may be read for key positions nobody holds. seq_start[i]: tokens sequence i held
 // before this step (its new keys are already in the cache). max_q_len: longest new run, for the grid.
-// scale must be positive. Options, each off at 0 / null: keep_first (with a window: the first keys of a sequence stay
+// scale must be positive. window: 0, n > 0 a sliding window, -n < 0 chunks of n positions (first_visible_key). Options,
+// each off at 0 / null: keep_first (with a window: the first keys of a sequence stay
 // visible behind it), sink (one more softmax term of score 0 without a value), gate (bfloat16 rows of n_q * hd
 // elements, gate_ld apart, 16-byte aligned: the output is multiplied by sigmoid(gate)).
 static int prefill_tc_entry(const void* q, const void* k_cache, const void* v_cache, void* out, const int* cu_q,
@@ -593,7 +596,7 @@ static int prefill_tc_entry(const void* q, const void* k_cache, const void* v_ca
                             const ScoreOptions so, cudaStream_t stream) {
   if (n_tokens < 0 || n_seqs < 0 || n_q <= 0 || n_kv <= 0 || n_q % n_kv || max_pages <= 0 || n_pages_total <= 0)
     return LLMIE_ERR_BAD_ARG;
-  if (keep_first < 0 || (gate && (gate_ld < n_q * hd || gate_ld % 8 || !aligned16(gate)))) return LLMIE_ERR_BAD_ARG;
+  if (keep_first < 0 || (window < 0 && keep_first) || (gate && (gate_ld < n_q * hd || gate_ld % 8 || !aligned16(gate)))) return LLMIE_ERR_BAD_ARG;
   if (!(scale > 0.f)) return LLMIE_ERR_BAD_ARG;   // the running maximum is taken before the scores are scaled
   if (so.softcap < 0.f || (so.dist_bias && so.bias_len <= 0) || (so.sink_vals && !sink)) return LLMIE_ERR_BAD_ARG;
   if (so.sigmoid_bias && (so.softcap > 0.f || so.dist_bias || so.sink_vals || sink)) return LLMIE_ERR_BAD_ARG;

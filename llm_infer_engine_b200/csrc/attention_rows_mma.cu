@@ -36,7 +36,7 @@ struct RowsArgs {
   const int* block_table;
   int max_pages, page_size, n_q, n_kv, hd, hdv, v_ld;
   float scale;
-  int window;
+  int window;                    // 0, n > 0 a sliding window, -n < 0 chunks of n positions (first_visible_key)
   float softcap;
   const float* dist_bias;        // [n_q, bias_len] or null
   int bias_len;
@@ -91,7 +91,7 @@ attention_rows_mma_kernel(const RowsArgs p) {
   const int tok_first = r0 / G;
   const int tok_last = min(r0 + kRmRows - 1, n_rows - 1) / G;
   const int pos_last = start + tok_last;
-  const int key_lo = p.window > 0 ? max(start + tok_first - p.window + 1, 0) : 0;
+  const int key_lo = first_visible_key(start + tok_first, p.window);
   const int tile_lo = key_lo / kRmKeys, tile_hi = pos_last / kRmKeys;
 
   // ---- the queries of the block's rows
@@ -132,6 +132,7 @@ attention_rows_mma_kernel(const RowsArgs p) {
   const int sm_row = warp * 4 + (lane >> 3), sm_key0 = (lane & 7) * 4;
   float m_run = -INFINITY, l_run = 0.f;
   const int pos_row = r0 + sm_row < n_rows ? start + (r0 + sm_row) / G : -1;
+  const int lo_row = pos_row >= 0 ? first_visible_key(pos_row, p.window) : 0;
   const float* bias_row = (p.dist_bias && r0 + sm_row < n_rows)
                               ? p.dist_bias + (size_t)(hk * G + (r0 + sm_row) % G) * p.bias_len : nullptr;
   float acc[2][NTW][4];
@@ -195,9 +196,10 @@ attention_rows_mma_kernel(const RowsArgs p) {
         const int col = sm_row * 33 + sm_key0 + e;
         float x = ((S[col] + S[kRmRows * 33 + col]) + (S[2 * kRmRows * 33 + col] + S[3 * kRmRows * 33 + col])) * p.scale;
         if (p.softcap > 0.f) x = p.softcap * rm_tanh(x * inv_cap);
-        const int dist = pos_row - (tile * kRmKeys + sm_key0 + e);
+        const int key = tile * kRmKeys + sm_key0 + e;
+        const int dist = pos_row - key;
         if (bias_row) x += bias_row[min(max(dist, 0), p.bias_len - 1)];
-        vis[e] = dist >= 0 && (p.window == 0 || dist < p.window);
+        vis[e] = dist >= 0 && key >= lo_row;
         sc[e] = vis[e] ? x : -INFINITY;
         mx = fmaxf(mx, sc[e]);
       }
@@ -335,7 +337,7 @@ extern "C" int llmie_attention_rows_mma(const void* q, const void* k_cache, cons
                                         const float* sink_vals, int sink, const float* sig_bias,
                                         cudaStream_t stream) {
   if (sig_bias && (sink || softcap > 0.f || dist_bias)) return LLMIE_ERR_BAD_ARG;
-  if (n_seqs < 0 || max_q_len < 0 || n_q <= 0 || n_kv <= 0 || n_q % n_kv || max_pages <= 0 || window < 0 || softcap < 0.f)
+  if (n_seqs < 0 || max_q_len < 0 || n_q <= 0 || n_kv <= 0 || n_q % n_kv || max_pages <= 0 || softcap < 0.f)
     return LLMIE_ERR_BAD_ARG;
   if ((dist_bias && bias_len <= 0) || (sink_vals && !sink) || v_ld < hdv) return LLMIE_ERR_BAD_ARG;
   if (!llmie_attention_rows_mma_supported(hd, hdv, page_size, shared_rows)) return LLMIE_ERR_UNSUPPORTED_SIZE;

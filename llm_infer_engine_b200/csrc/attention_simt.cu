@@ -8,7 +8,8 @@
 // h reading key/value head h / (Hq / Hkv).
 //
 // A token at absolute position p of its sequence sees keys lo..p of that sequence's slot,
-// lo = max(0, p - window + 1) when window > 0, else 0, and besides them the first `keep_first` keys of the
+// lo = max(0, p - window + 1) when window > 0, the start of p's chunk of -window positions when window < 0 (chunks
+// counted from position 0), else 0, and besides them the first `keep_first` keys of the
 // sequence (keys 0..keep_first-1 stay visible when the window has moved past them). Keys of this very step were
 // written to the cache before this kernel runs, so prefill at any start position, decode, and mixtures need
 // no separate code.
@@ -50,7 +51,7 @@ attention_paged_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
   const int pos = tok_pos[t];
   const int slot = seq_slot[tok_seq[t]];
   const int* pages = block_table + (size_t)slot * max_pages;
-  const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+  const int lo = first_visible_key(pos, window);
   const int kept = keep_first < lo ? keep_first : lo;     // keys [0, kept) are seen besides [lo, pos]
 
   float* qs = q_smem + warp * hd;
@@ -181,7 +182,7 @@ extern "C" int llmie_attention_paged_sig(const void* q, const void* k_cache, con
   if (sig_bias && sink) return LLMIE_ERR_BAD_ARG;
   if (n_tokens < 0 || n_q <= 0 || n_kv <= 0 || hd <= 0 || hdv <= 0 || page_size <= 0 || max_pages <= 0)
     return LLMIE_ERR_BAD_ARG;
-  if (n_q % n_kv || keep_first < 0 || window < 0 || (gate && gate_ld < n_q * hdv)) return LLMIE_ERR_BAD_ARG;
+  if (n_q % n_kv || keep_first < 0 || (window < 0 && keep_first) || (gate && gate_ld < n_q * hdv)) return LLMIE_ERR_BAD_ARG;
   if (v_ld < hdv || softcap < 0.f || (dist_bias && bias_len <= 0) || (sink_vals && !sink)) return LLMIE_ERR_BAD_ARG;
   if (hd > kWideHeadDim || hdv > kWideHeadDim) return LLMIE_ERR_UNSUPPORTED_SIZE;
   if (dtype != LLMIE_F32 && dtype != LLMIE_BF16) return LLMIE_ERR_DTYPE;

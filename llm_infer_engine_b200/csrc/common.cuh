@@ -101,6 +101,15 @@ __device__ __forceinline__ float apply_act(float z, int act) {
   }
 }
 
+// The first key a token at position `pos` may see, by the `window` argument of the attention kernels: 0 = every earlier
+// key; n > 0 = the last n keys, its own included; -n < 0 = the keys of its own chunk of n positions (chunks counted from
+// position 0 of the sequence).
+__device__ __forceinline__ int first_visible_key(int pos, int window) {
+  if (window > 0) return max(pos - window + 1, 0);
+  if (window < 0) return pos - pos % -window;
+  return 0;
+}
+
 static inline bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; }
 
 // Programmatic dependent launch: a kernel launched through launch_k may begin while the kernel

@@ -194,7 +194,7 @@ skinny_gemm_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __r
       const size_t o = (size_t)b * ldo + n;
       if (EPI == kStoreBf16) reinterpret_cast<__nv_bfloat16*>(out)[o] = __float2bfloat16_rn(v);
       if (EPI == kStoreF32) reinterpret_cast<float*>(out)[o] = v;
-      if (EPI == kAddF32) reinterpret_cast<float*>(out)[o] += v;
+      if (EPI == kAddF32) reinterpret_cast<float*>(out)[o] += bias ? v + bias[n] : v;
       if (EPI == kBiasAct)
         reinterpret_cast<__nv_bfloat16*>(out)[o] = __float2bfloat16_rn(apply_act(bias ? v + bias[n] : v, act));
     }
@@ -289,6 +289,12 @@ extern "C" int llmie_gemm_skinny_gated(const void* x, const void* W, void* out, 
                                        cudaStream_t stream) {
   if (act < 0 || act > 4) return LLMIE_ERR_BAD_ARG;
   return gemm_skinny_entry(x, W, out, batch, N, K, ldo, kSwiGLU, nullptr, act == 4 ? 0 : act, stream);
+}
+
+// out float32 [batch, ldo] += x W^T + bias (bias float32 [N] or null).
+extern "C" int llmie_gemm_skinny_add_bias(const void* x, const void* W, void* out, int batch, int N, int K, int ldo,
+                                          const float* bias, cudaStream_t stream) {
+  return gemm_skinny_entry(x, W, out, batch, N, K, ldo, kAddF32, bias, 0, stream);
 }
 
 // out bfloat16 [batch, ldo] = act(x W^T + bias) in one kernel.

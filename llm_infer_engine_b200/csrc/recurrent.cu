@@ -10,11 +10,14 @@
 //   matrix_gates       q = silu(q_raw), f = l + (1 - l) sigmoid(f_raw + b)           element-wise, float32 out
 //   matrix_scan        S <- diag(f_t) S + (1 - f_t) v_t^T ; o_t = S^T q_t            S [dim, vdim] per head
 //                      keyed form (a decay per head given): S <- a_h S + k_t v_t^T   linear attention with a constant decay
+//                      stepped form (a decay and a factor per token and head): S <- a_t S + (c_t k_t) v_t^T, keys and
+//                      queries shared by groups of heads (a state space model)
 //   act_columns        float32 copies of up to three runs of columns of the projections, through an activation
 //   matrix_scan_chunked  the same for long pieces, cut into chunks that run side by side (below)
 //   head_rmsnorm       o / sqrt(mean(o^2) + eps) * w over each head's vdim (or over the whole row, with a weight per
 //                      column), optionally times sigmoid(gate)
-//   causal_conv        u_t = b + sum_j taps[:, K-1-j] x_(t-j), x before the step from the state's last K-1 inputs
+//   causal_conv        u_t = act(b + sum_j taps[:, K-1-j] x_(t-j)), x before the step from the state's last K-1 inputs
+//   conv_state_store   the last K-1 inputs after the step (a one-token step's causal_conv writes them itself)
 //   unit_gate_values   a = exp(-c r softplus(lam)), drive = sqrt(1 - a^2) i u, r and i sigmoids of given pre-activations
 //   unit_scan          S <- a_t S + drive_t ; out_t = S act(y_raw + b) ; the new conv state
 //   unit_scan_chunked  the same for long pieces, 32 chunks of a sequence side by side in one block
@@ -62,23 +65,25 @@ constexpr int kScanRWide = 8;       // ... when it owns four columns
 // bits), R = ceil(dim / S) <= RMAX. With four columns a thread every gate, key and query entry that is loaded serves
 // four state entries: the kernel is bound by what the first-level cache delivers otherwise. The next token's gate, query
 // and values are requested before the current token's products.
-// With `head_decay` (float32 [H]) the update is S <- head_decay[h] S + k_t v_t^T with the keys k_t in the place of fg.
+// FORM 1 (keyed): with `head_decay` (float32 [H]) the update is S <- head_decay[h] S + k_t v_t^T with the keys k_t in the
+// place of fg. FORM 2 (stepped): head_decay and key_factor are float32 [T, H], S <- head_decay[t, h] S + (key_factor[t, h]
+// k_t) v_t^T, and qa and fg have G <= H heads, each shared by H / G heads of the state. FORM 0: fg holds gates, G = H.
 // MODE 0: a sequence's whole piece, from the slot's state to the slot's state. MODE 1 and 2 work on chunk c =
 // blockIdx.z % NC of sequence blockIdx.z / NC, L tokens each, with ws float32 [n_seqs, NC, H, D, Dv] and decay float32
 // [n_seqs, NC, H, D]: MODE 1 runs a chunk that is not the sequence's last from a zero state, without outputs, and leaves
 // its end state in ws[c + 1] and the product of its gates in decay[c + 1]; MODE 2 runs a chunk from ws[c] with outputs,
 // and the last one writes the slot's state.
-template <typename T, int MODE, int C, int RMAX, bool KEYED>
+template <typename T, int MODE, int C, int RMAX, int FORM>
 __global__ void __launch_bounds__(kScanThreads)
 matrix_scan_kernel(const float* __restrict__ qa, const float* __restrict__ fg, const T* __restrict__ v, int v_ld,
                    float* __restrict__ state, const int* __restrict__ cu_q, const int* __restrict__ seq_slot,
                    float* __restrict__ o, int H, int D, int Dv, int S, int R, int write_state,
                    float* __restrict__ ws, float* __restrict__ decay, int L, int NC,
-                   const float* __restrict__ head_decay) {
+                   const float* __restrict__ head_decay, const float* __restrict__ key_factor, int G) {
   pdl_launch_dependents();
-  // keyed form: fg holds keys k_t instead of gates, and the gate of every row of head h is the constant head_decay[h]
-  constexpr bool keyed = KEYED;
-  const float dh = keyed ? head_decay[blockIdx.y] : 0.f;       // a constant of the model: no kernel writes it
+  // keyed forms: fg holds keys k_t instead of gates, and every row of head h has the same gate
+  constexpr bool keyed = FORM != 0, stepped = FORM == 2;
+  const float dh = FORM == 1 ? head_decay[blockIdx.y] : 0.f;   // a constant of the model: no kernel writes it
   pdl_wait();
   const int s = threadIdx.x & (S - 1);
   const int col = threadIdx.x / S;
@@ -105,10 +110,16 @@ matrix_scan_kernel(const float* __restrict__ qa, const float* __restrict__ fg, c
     for (int c = 0; c < C; ++c)
       St[r][c] = (MODE != 1 && r < R && i0 + r < D) ? start[(size_t)(i0 + r) * Dv + c] : 0.f;
   float f[RMAX], q[RMAX], vj[C];
-  const size_t HD = (size_t)H * D;
+  const size_t HD = (size_t)G * D;
+  const int hq = stepped ? h / (H / G) : h;
+  float dt_gate = 0.f, dt_factor = 0.f;             // stepped form: the next token's decay and key factor
   auto fetch = [&](int t) {
-    const float* fr = fg + (size_t)t * HD + (size_t)h * D + i0;
-    const float* qr = qa + (size_t)t * HD + (size_t)h * D + i0;
+    const float* fr = fg + (size_t)t * HD + (size_t)hq * D + i0;
+    const float* qr = qa + (size_t)t * HD + (size_t)hq * D + i0;
+    if (stepped) {
+      dt_gate = head_decay[(size_t)t * H + h];
+      dt_factor = key_factor[(size_t)t * H + h];
+    }
 #pragma unroll
     for (int r = 0; r < RMAX; ++r) {
       const bool ok = r < R && i0 + r < D;
@@ -128,11 +139,12 @@ matrix_scan_kernel(const float* __restrict__ qa, const float* __restrict__ fg, c
     for (int c = 0; c < C; ++c) { cv[c] = vj[c]; acc[c] = 0.f; }
 #pragma unroll
     for (int r = 0; r < RMAX; ++r) { cf[r] = f[r]; cq[r] = MODE != 1 ? q[r] : 0.f; }
+    const float tg = dt_gate, tf = dt_factor;
     if (t + 1 < t1) fetch(t + 1);
 #pragma unroll
     for (int r = 0; r < RMAX; ++r) {
-      const float gate = keyed ? dh : cf[r];
-      const float write = keyed ? cf[r] : 1.f - cf[r];
+      const float gate = stepped ? tg : (keyed ? dh : cf[r]);
+      const float write = stepped ? tf * cf[r] : (keyed ? cf[r] : 1.f - cf[r]);
 #pragma unroll
       for (int c = 0; c < C; ++c) {
         St[r][c] = fmaf(gate, St[r][c], write * cv[c]);
@@ -300,24 +312,48 @@ __global__ void act_columns_kernel(const T* __restrict__ proj, int ld, int off0,
 // ------------------------------------------------------------------------------------------ vector state
 constexpr int kMaxTaps = 16;
 
-// A thread is a channel over a run of `tile` consecutive packed tokens. x = proj[:, x_off + c] + x_bias; inputs before
-// the step come from conv_state [slots, K-1, C] (the last K-1 inputs of the sequence so far, zeros at its start). The
-// thread keeps the last K inputs in registers: a token that follows its predecessor in the same sequence loads ONE new
+// A thread is V adjacent channels over a run of `tile` consecutive packed tokens. x = proj[:, x_off + c] + x_bias; inputs
+// before the step come from conv_state [slots, K-1, C] (the last K-1 inputs of the sequence so far, zeros at its start).
+// The thread keeps the last K inputs in registers: a token that follows its predecessor in the same sequence loads ONE new
 // input, the first token of a run or of a sequence's piece loads all K. Oldest input first: a fixed order of summation.
-template <typename T>
-__global__ void causal_conv_kernel(const T* __restrict__ proj, int ld, int x_off, const float* __restrict__ x_bias,
-                                   const float* __restrict__ taps, const float* __restrict__ conv_bias,
-                                   const float* __restrict__ conv_state, const int* __restrict__ cu_q,
-                                   const int* __restrict__ tok_seq, const int* __restrict__ seq_slot,
-                                   float* __restrict__ u, int C, int K, int n_tokens, int tile) {
-  pdl_launch_dependents();
-  const int c = blockIdx.x * blockDim.x + threadIdx.x;
-  if (c >= C) return;
-  float tp[kMaxTaps], w[kMaxTaps];
+// `act`: an activation of the result. `single`: every sequence of the step brings one token, so a channel's inputs are
+// this thread's alone and it also writes the new conv_state (in other steps conv_state_store does).
+template <typename TP, int V>
+__device__ __forceinline__ void conv_input(const TP* p, const float (&xb)[V], float (&x)[V]) {
+  if (V == 4) {
+    if (sizeof(TP) == 4) {
+      const float4 r = *reinterpret_cast<const float4*>(p);
+      x[0] = r.x; x[1 % V] = r.y; x[2 % V] = r.z; x[3 % V] = r.w;
+    } else {
+      const uint2 r = *reinterpret_cast<const uint2*>(p);
+      const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x));
+      const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
+      x[0] = lo.x; x[1 % V] = lo.y; x[2 % V] = hi.x; x[3 % V] = hi.y;
+    }
+  } else {
+    x[0] = to_f32(p[0]);
+  }
 #pragma unroll
-  for (int k = 0; k < kMaxTaps; ++k) tp[k] = k < K ? taps[(size_t)c * K + k] : 0.f;       // weights: no kernel writes them
-  const float xb = x_bias ? x_bias[c] : 0.f;
-  const float cb = conv_bias ? conv_bias[c] : 0.f;
+  for (int e = 0; e < V; ++e) x[e] += xb[e];
+}
+
+template <typename TP, typename TO, int KM, int V>
+__global__ void causal_conv_kernel(const TP* __restrict__ proj, int ld, int x_off, const float* __restrict__ x_bias,
+                                   const float* __restrict__ taps, const float* __restrict__ conv_bias,
+                                   float* conv_state, const int* __restrict__ cu_q,
+                                   const int* __restrict__ tok_seq, const int* __restrict__ seq_slot,
+                                   TO* __restrict__ u, int C, int K, int n_tokens, int tile, int act, int single) {
+  pdl_launch_dependents();
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (c >= C) return;
+  float tp[KM][V], w[KM][V], xb[V], cb[V];
+#pragma unroll
+  for (int e = 0; e < V; ++e) {
+#pragma unroll
+    for (int k = 0; k < KM; ++k) tp[k][e] = k < K ? taps[(size_t)(c + e) * K + k] : 0.f;   // weights: no kernel writes them
+    xb[e] = x_bias ? x_bias[c + e] : 0.f;
+    cb[e] = conv_bias ? conv_bias[c + e] : 0.f;
+  }
   pdl_wait();
   const int ta = blockIdx.y * tile, tb = min(ta + tile, n_tokens);
   int prev_seq = -1;
@@ -327,29 +363,92 @@ __global__ void causal_conv_kernel(const T* __restrict__ proj, int ld, int x_off
     if (seq != prev_seq || p == 0) {
       const float* old = conv_state + (size_t)seq_slot[seq] * (K - 1) * C + c;
 #pragma unroll
-      for (int k = 0; k < kMaxTaps; ++k) {
+      for (int k = 0; k < KM; ++k) {
         if (k < K) {
           const int m = p - (K - 1 - k);              // w[k] is the input K-1-k tokens back
-          w[k] = m >= 0 ? to_f32(proj[(size_t)(t - (K - 1 - k)) * ld + x_off + c]) + xb
-                        : old[(size_t)(K - 1 + m) * C];
+          if (m >= 0) {
+            conv_input<TP, V>(proj + (size_t)(t - (K - 1 - k)) * ld + x_off + c, xb, w[k]);
+          } else {
+#pragma unroll
+            for (int e = 0; e < V; ++e) w[k][e] = old[(size_t)(K - 1 + m) * C + e];
+          }
         }
       }
       prev_seq = seq;
     } else {
 #pragma unroll
-      for (int k = 0; k + 1 < kMaxTaps; ++k)
-        if (k + 1 < K) w[k] = w[k + 1];
-      const float x = to_f32(proj[(size_t)t * ld + x_off + c]) + xb;
+      for (int k = 0; k + 1 < KM; ++k)
+        if (k + 1 < K) {
 #pragma unroll
-      for (int k = 0; k < kMaxTaps; ++k)
-        if (k == K - 1) w[k] = x;
+          for (int e = 0; e < V; ++e) w[k][e] = w[k + 1][e];
+        }
+      float x[V];
+      conv_input<TP, V>(proj + (size_t)t * ld + x_off + c, xb, x);
+#pragma unroll
+      for (int k = 0; k < KM; ++k)
+        if (k == K - 1) {
+#pragma unroll
+          for (int e = 0; e < V; ++e) w[k][e] = x[e];
+        }
     }
-    float acc = cb;
+    float acc[V];
 #pragma unroll
-    for (int k = 0; k < kMaxTaps; ++k)
-      if (k < K) acc = fmaf(tp[k], w[k], acc);
-    u[(size_t)t * C + c] = acc;
+    for (int e = 0; e < V; ++e) {
+      acc[e] = cb[e];
+#pragma unroll
+      for (int k = 0; k < KM; ++k)
+        if (k < K) acc[e] = fmaf(tp[k][e], w[k][e], acc[e]);
+      acc[e] = apply_act(acc[e], act);
+    }
+    TO* dst = u + (size_t)t * C + c;
+    if (V == 4 && sizeof(TO) == 4) {
+      *reinterpret_cast<float4*>(dst) = make_float4(acc[0], acc[1 % V], acc[2 % V], acc[3 % V]);
+    } else if (V == 4) {
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(acc[0], acc[1 % V]), hi = __floats2bfloat162_rn(acc[2 % V], acc[3 % V]);
+      uint2 raw;
+      raw.x = *reinterpret_cast<const unsigned*>(&lo);
+      raw.y = *reinterpret_cast<const unsigned*>(&hi);
+      *reinterpret_cast<uint2*>(dst) = raw;
+    } else {
+      dst[0] = from_f32<TO>(acc[0]);
+    }
+    if (single) {
+      float* cs = conv_state + (size_t)seq_slot[seq] * (K - 1) * C + c;
+#pragma unroll
+      for (int k = 0; k + 1 < KM; ++k)
+        if (k + 1 < K) {
+#pragma unroll
+          for (int e = 0; e < V; ++e) cs[(size_t)k * C + e] = w[k + 1][e];
+        }
+    }
   }
+}
+
+// The convolution's new state: a thread per (sequence, channel) leaves the last K-1 inputs of the sequence, this step's
+// and before them what the state held.
+template <typename T>
+__global__ void conv_state_store_kernel(const T* __restrict__ proj, int ld, int x_off, const float* __restrict__ x_bias,
+                                        float* __restrict__ conv_state, const int* __restrict__ cu_q,
+                                        const int* __restrict__ seq_slot, int C, int K) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  const int seq = blockIdx.y;
+  if (c >= C) return;
+  const int t0 = cu_q[seq], n = cu_q[seq + 1] - t0;
+  float* cs = conv_state + (size_t)seq_slot[seq] * (K - 1) * C + c;
+  const float xb = x_bias ? x_bias[c] : 0.f;
+  float keep[kMaxTaps];
+#pragma unroll
+  for (int k = 0; k < kMaxTaps; ++k) {
+    if (k < K - 1) {
+      const int m = n - (K - 1) + k;                  // place within the step, negative = before it
+      keep[k] = m >= 0 ? to_f32(proj[(size_t)(t0 + m) * ld + x_off + c]) + xb : cs[(size_t)(K - 1 + m) * C];
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < kMaxTaps; ++k)
+    if (k < K - 1) cs[(size_t)k * C] = keep[k];
 }
 
 // gates [T, groups * 2 * bw]: per group the pre-activations of r (bw) and then of i (bw). In place: r's place receives
@@ -565,104 +664,101 @@ extern "C" int llmie_matrix_gates(const void* proj, int ld, int q_off, int f_off
   return LLMIE_OK;
 }
 
+// What one of the scans reads and writes, whatever its form.
+struct ScanArgs {
+  const float* qa;
+  const float* fg;
+  const void* v;
+  int v_ld;
+  float* state;
+  const int* cu_q;
+  const int* seq_slot;
+  float* o;
+  int n_seqs, H, D, Dv, write_state;
+  const float* head_decay;     // FORM 1: [H], FORM 2: [T, H], FORM 0: null
+  const float* key_factor;     // FORM 2: [T, H], else null
+  int G;                       // heads of qa and fg
+  float* ws;                   // chunked: scratch, else null
+  float* decay;
+  int chunk, n_chunks;
+};
+
+template <typename T, int C, int RM, int FORM>
+static void matrix_scan_launch(const ScanArgs& a, const ScanShape& g, cudaStream_t stream) {
+  const int cols = (kScanThreads / g.S) * C;
+  const bool chunked = a.ws != nullptr;
+  const dim3 grid((a.Dv + cols - 1) / cols, a.H, a.n_seqs * (chunked ? a.n_chunks : 1)), block(kScanThreads);
+#define LLMIE_SCAN_ARGS                                                                                                   \
+  grid, block, 0, stream, a.qa, a.fg, (const T*)a.v, a.v_ld, a.state, a.cu_q, a.seq_slot, a.o, a.H, a.D, a.Dv, g.S, g.R, \
+      a.write_state, a.ws, a.decay, a.chunk, a.n_chunks, a.head_decay, a.key_factor, a.G
+  if (!chunked) {
+    launch_k(matrix_scan_kernel<T, 0, C, RM, FORM>, LLMIE_SCAN_ARGS);
+    return;
+  }
+  launch_k(matrix_scan_kernel<T, 1, C, RM, FORM>, LLMIE_SCAN_ARGS);
+  const size_t HDDv = (size_t)a.H * a.D * a.Dv;
+  launch_k(matrix_scan_chain_kernel, dim3((unsigned)((HDDv + 255) / 256), a.n_seqs), dim3(256), 0, stream,
+           (const float*)a.state, a.cu_q, a.seq_slot, a.ws, (const float*)a.decay, a.H, a.D, a.Dv, a.chunk, a.n_chunks);
+  launch_k(matrix_scan_kernel<T, 2, C, RM, FORM>, LLMIE_SCAN_ARGS);
+#undef LLMIE_SCAN_ARGS
+}
+
+template <int FORM>
+static int matrix_scan_entry(const ScanArgs& a, int dtype, cudaStream_t stream) {
+  if (a.n_seqs < 0 || a.H <= 0 || a.D <= 0 || a.Dv <= 0 || a.v_ld < a.H * a.Dv || a.G <= 0 || a.H % a.G)
+    return LLMIE_ERR_BAD_ARG;
+  if (a.ws && (a.chunk <= 0 || a.n_chunks <= 0 || !a.decay)) return LLMIE_ERR_BAD_ARG;
+  if (a.D > 32 * kScanR) return LLMIE_ERR_UNSUPPORTED_SIZE;
+  if (a.n_seqs == 0) return LLMIE_OK;
+  if (a.H > 65535 || a.n_seqs > 65535 || (a.ws && (long long)a.n_seqs * a.n_chunks > 65535)) return LLMIE_ERR_UNSUPPORTED_SIZE;
+  const ScanShape g = scan_shape(a.D, a.Dv);
+  if (dtype == LLMIE_F32) {
+    if (g.C == 4) matrix_scan_launch<float, 4, kScanRWide, FORM>(a, g, stream);
+    else matrix_scan_launch<float, 1, kScanR, FORM>(a, g, stream);
+  } else if (dtype == LLMIE_BF16) {
+    if (g.C == 4) matrix_scan_launch<__nv_bfloat16, 4, kScanRWide, FORM>(a, g, stream);
+    else matrix_scan_launch<__nv_bfloat16, 1, kScanR, FORM>(a, g, stream);
+  } else {
+    return LLMIE_ERR_DTYPE;
+  }
+  LLMIE_LAUNCH_CHECK();
+  return LLMIE_OK;
+}
+
 // qa, fg float32 [T, H * D]; v rows of H * Dv elements of `dtype`, v_ld apart; state float32 [slots, H, D, Dv];
 // o float32 [T, H * Dv]. D up to 512.
 // head_decay float32 [H] or null: with it, fg holds keys and S <- head_decay[h] S + k_t v_t^T.
 extern "C" int llmie_matrix_scan_ex(const float* qa, const float* fg, const void* v, int v_ld, float* state,
                                     const int* cu_q, const int* seq_slot, float* o, int n_seqs, int H, int D, int Dv,
                                     int write_state, int dtype, const float* head_decay, cudaStream_t stream) {
-  if (n_seqs < 0 || H <= 0 || D <= 0 || Dv <= 0 || v_ld < H * Dv) return LLMIE_ERR_BAD_ARG;
-  if (D > 32 * kScanR) return LLMIE_ERR_UNSUPPORTED_SIZE;
-  if (n_seqs == 0) return LLMIE_OK;
-  const ScanShape g = scan_shape(D, Dv);
-  const int S = g.S, R = g.R;
-  const int cols = (kScanThreads / S) * g.C;
-  const dim3 grid((Dv + cols - 1) / cols, H, n_seqs), block(kScanThreads);
-  if (grid.y > 65535 || grid.z > 65535) return LLMIE_ERR_UNSUPPORTED_SIZE;
-#define LLMIE_SCAN0_(T, C, RM, K)                                                                                           \
-  launch_k(matrix_scan_kernel<T, 0, C, RM, K>, grid, block, 0, stream, qa, fg, (const T*)v, v_ld, state, cu_q, seq_slot, o, \
-           H, D, Dv, S, R, write_state, (float*)nullptr, (float*)nullptr, 0, 1, head_decay)
-#define LLMIE_SCAN0(T, C, RM)                                      \
-  do {                                                             \
-    if (head_decay) LLMIE_SCAN0_(T, C, RM, true);                  \
-    else LLMIE_SCAN0_(T, C, RM, false);                            \
-  } while (0)
-  if (dtype == LLMIE_F32) {
-    if (g.C == 4) LLMIE_SCAN0(float, 4, kScanRWide); else LLMIE_SCAN0(float, 1, kScanR);
-  } else if (dtype == LLMIE_BF16) {
-    if (g.C == 4) LLMIE_SCAN0(__nv_bfloat16, 4, kScanRWide); else LLMIE_SCAN0(__nv_bfloat16, 1, kScanR);
-  } else {
-    return LLMIE_ERR_DTYPE;
-  }
-#undef LLMIE_SCAN0
-#undef LLMIE_SCAN0_
-  LLMIE_LAUNCH_CHECK();
-  return LLMIE_OK;
+  const ScanArgs a{qa, fg, v, v_ld, state, cu_q, seq_slot, o, n_seqs, H, D, Dv, write_state, head_decay, nullptr, H,
+                   nullptr, nullptr, 0, 1};
+  return head_decay ? matrix_scan_entry<1>(a, dtype, stream) : matrix_scan_entry<0>(a, dtype, stream);
 }
 
-extern "C" int llmie_matrix_scan(const float* qa, const float* fg, const void* v, int v_ld, float* state,
-                                 const int* cu_q, const int* seq_slot, float* o, int n_seqs, int H, int D, int Dv,
-                                 int write_state, int dtype, cudaStream_t stream) {
-  return llmie_matrix_scan_ex(qa, fg, v, v_ld, state, cu_q, seq_slot, o, n_seqs, H, D, Dv, write_state, dtype, nullptr,
-                              stream);
-}
-
-template <typename T, int C, int RM, bool K>
-static void matrix_scan_chunked_launch(const float* qa, const float* fg, const T* v, int v_ld, float* state,
-                                       const int* cu_q, const int* seq_slot, float* o, float* ws, float* decay,
-                                       int n_seqs, int H, int D, int Dv, int S, int R, int L, int NC, int write_state,
-                                       const float* head_decay, cudaStream_t stream) {
-  const int cols = (kScanThreads / S) * C;
-  const dim3 grid((Dv + cols - 1) / cols, H, n_seqs * NC), block(kScanThreads);
-  launch_k(matrix_scan_kernel<T, 1, C, RM, K>, grid, block, 0, stream, qa, fg, v, v_ld, state, cu_q, seq_slot, o, H, D, Dv, S, R,
-           write_state, ws, decay, L, NC, head_decay);
-  const size_t HDDv = (size_t)H * D * Dv;
-  launch_k(matrix_scan_chain_kernel, dim3((unsigned)((HDDv + 255) / 256), n_seqs), dim3(256), 0, stream,
-           (const float*)state, cu_q, seq_slot, ws, (const float*)decay, H, D, Dv, L, NC);
-  launch_k(matrix_scan_kernel<T, 2, C, RM, K>, grid, block, 0, stream, qa, fg, v, v_ld, state, cu_q, seq_slot, o, H, D, Dv, S, R,
-           write_state, ws, decay, L, NC, head_decay);
-}
-
-// llmie_matrix_scan for long pieces: chunks of `chunk` tokens run side by side. n_chunks >= ceil(longest piece / chunk);
-// ws float32 [n_seqs, n_chunks, H, D, Dv] and decay float32 [n_seqs, n_chunks, H, D] are scratch.
+// llmie_matrix_scan_ex for long pieces: chunks of `chunk` tokens run side by side. n_chunks >= ceil(longest piece /
+// chunk); ws float32 [n_seqs, n_chunks, H, D, Dv] and decay float32 [n_seqs, n_chunks, H, D] are scratch.
 extern "C" int llmie_matrix_scan_chunked_ex(const float* qa, const float* fg, const void* v, int v_ld, float* state,
                                             const int* cu_q, const int* seq_slot, float* o, float* ws, float* decay,
                                             int n_seqs, int H, int D, int Dv, int chunk, int n_chunks, int write_state,
                                             int dtype, const float* head_decay, cudaStream_t stream) {
-  if (n_seqs < 0 || H <= 0 || D <= 0 || Dv <= 0 || v_ld < H * Dv || chunk <= 0 || n_chunks <= 0 || !ws || !decay)
-    return LLMIE_ERR_BAD_ARG;
-  if (D > 32 * kScanR) return LLMIE_ERR_UNSUPPORTED_SIZE;
-  if (n_seqs == 0) return LLMIE_OK;
-  const ScanShape g = scan_shape(D, Dv);
-  const int S = g.S, R = g.R;
-  if (H > 65535 || (long long)n_seqs * n_chunks > 65535 || n_seqs > 65535) return LLMIE_ERR_UNSUPPORTED_SIZE;
-#define LLMIE_SCANC_(T, C, RM, K)                                                                                            \
-  matrix_scan_chunked_launch<T, C, RM, K>(qa, fg, (const T*)v, v_ld, state, cu_q, seq_slot, o, ws, decay, n_seqs, H, D, Dv, \
-                                          S, R, chunk, n_chunks, write_state, head_decay, stream)
-#define LLMIE_SCANC(T, C, RM)                                      \
-  do {                                                             \
-    if (head_decay) LLMIE_SCANC_(T, C, RM, true);                  \
-    else LLMIE_SCANC_(T, C, RM, false);                            \
-  } while (0)
-  if (dtype == LLMIE_F32) {
-    if (g.C == 4) LLMIE_SCANC(float, 4, kScanRWide); else LLMIE_SCANC(float, 1, kScanR);
-  } else if (dtype == LLMIE_BF16) {
-    if (g.C == 4) LLMIE_SCANC(__nv_bfloat16, 4, kScanRWide); else LLMIE_SCANC(__nv_bfloat16, 1, kScanR);
-  } else {
-    return LLMIE_ERR_DTYPE;
-  }
-#undef LLMIE_SCANC
-#undef LLMIE_SCANC_
-  LLMIE_LAUNCH_CHECK();
-  return LLMIE_OK;
+  if (!ws || !decay) return LLMIE_ERR_BAD_ARG;
+  const ScanArgs a{qa, fg, v, v_ld, state, cu_q, seq_slot, o, n_seqs, H, D, Dv, write_state, head_decay, nullptr, H,
+                   ws, decay, chunk, n_chunks};
+  return head_decay ? matrix_scan_entry<1>(a, dtype, stream) : matrix_scan_entry<0>(a, dtype, stream);
 }
 
-extern "C" int llmie_matrix_scan_chunked(const float* qa, const float* fg, const void* v, int v_ld, float* state,
+// The stepped form: qa (queries) and fg (keys) float32 [T, G * D], shared by H / G heads each; decay and factor per token
+// and head, float32 [T, H]: S <- token_decay S + (key_factor k) v^T. ws null: unchunked, else as above.
+extern "C" int llmie_matrix_scan_stepped(const float* qa, const float* fg, const void* v, int v_ld, float* state,
                                          const int* cu_q, const int* seq_slot, float* o, float* ws, float* decay,
-                                         int n_seqs, int H, int D, int Dv, int chunk, int n_chunks, int write_state,
-                                         int dtype, cudaStream_t stream) {
-  return llmie_matrix_scan_chunked_ex(qa, fg, v, v_ld, state, cu_q, seq_slot, o, ws, decay, n_seqs, H, D, Dv, chunk,
-                                      n_chunks, write_state, dtype, nullptr, stream);
+                                         int n_seqs, int H, int G, int D, int Dv, int chunk, int n_chunks,
+                                         int write_state, int dtype, const float* token_decay, const float* key_factor,
+                                         cudaStream_t stream) {
+  if (!token_decay || !key_factor) return LLMIE_ERR_BAD_ARG;
+  const ScanArgs a{qa, fg, v, v_ld, state, cu_q, seq_slot, o, n_seqs, H, D, Dv, write_state, token_decay, key_factor, G,
+                   ws, decay, chunk, n_chunks};
+  return matrix_scan_entry<2>(a, dtype, stream);
 }
 
 // proj [T, ld] of `dtype`; out_k float32 [T, n_k] = act(proj[:, off_k : off_k + n_k]) for up to three runs (n_k = 0: unused).
@@ -728,26 +824,62 @@ extern "C" int llmie_head_rmsnorm(const float* o, const float* w, float eps, voi
   return llmie_head_rmsnorm_gated(o, w, eps, y, n_items, Dv, dtype, nullptr, 0, 1, stream);
 }
 
+template <typename TP, typename TO>
+static void causal_conv_launch(const TP* proj, int ld, int x_off, const float* x_bias, const float* taps,
+                               const float* conv_bias, float* conv_state, const int* cu_q, const int* tok_seq,
+                               const int* seq_slot, TO* u, int n_tokens, int C, int K, int act, int single,
+                               cudaStream_t stream) {
+  const bool by4 = K <= 4 && C % 4 == 0 && ld % 4 == 0 && x_off % 4 == 0 && aligned16(proj) && aligned16(u);
+  const int tile = n_tokens >= 1024 ? 16 : (n_tokens >= 64 ? 4 : 1);
+  const int units = by4 ? C / 4 : C;
+  const int threads = units >= 128 ? 128 : ((units + 31) / 32) * 32;
+  const dim3 grid((units + threads - 1) / threads, (n_tokens + tile - 1) / tile), block(threads);
+  if (by4)
+    launch_k(causal_conv_kernel<TP, TO, 4, 4>, grid, block, 0, stream, proj, ld, x_off, x_bias, taps, conv_bias, conv_state,
+             cu_q, tok_seq, seq_slot, u, C, K, n_tokens, tile, act, single);
+  else
+    launch_k(causal_conv_kernel<TP, TO, kMaxTaps, 1>, grid, block, 0, stream, proj, ld, x_off, x_bias, taps, conv_bias,
+             conv_state, cu_q, tok_seq, seq_slot, u, C, K, n_tokens, tile, act, single);
+}
+
 // proj [T, ld] of `dtype` with the convolution's input at column x_off (C columns); x_bias, conv_bias float32 [C] or
 // null; taps float32 [C, K] (the last column multiplies the current token); conv_state float32 [slots, K-1, C];
-// u float32 [T, C].
-extern "C" int llmie_causal_conv(const void* proj, int ld, int x_off, const float* x_bias, const float* taps,
-                                 const float* conv_bias, const float* conv_state, const int* cu_q, const int* tok_seq,
-                                 const int* seq_slot, float* u, int n_tokens, int C, int K, int dtype,
-                                 cudaStream_t stream) {
-  if (n_tokens < 0 || C <= 0 || K <= 0 || x_off < 0 || ld < x_off + C) return LLMIE_ERR_BAD_ARG;
-  if (K > kMaxTaps) return LLMIE_ERR_UNSUPPORTED_SIZE;
+// u [T, C] of u_dtype = act(convolution), act a code of apply_act. single != 0: every sequence brings one token and the
+// new conv_state is written too.
+extern "C" int llmie_causal_conv_ex(const void* proj, int ld, int x_off, const float* x_bias, const float* taps,
+                                    const float* conv_bias, float* conv_state, const int* cu_q, const int* tok_seq,
+                                    const int* seq_slot, void* u, int u_dtype, int n_tokens, int C, int K, int act,
+                                    int single, int dtype, cudaStream_t stream) {
+  if (n_tokens < 0 || C <= 0 || K <= 0 || x_off < 0 || ld < x_off + C || act < 0 || act > 4) return LLMIE_ERR_BAD_ARG;
+  if (K > kMaxTaps || n_tokens > 65535 * 16) return LLMIE_ERR_UNSUPPORTED_SIZE;
   if (n_tokens == 0) return LLMIE_OK;
-  const int tile = n_tokens >= 1024 ? 16 : (n_tokens >= 64 ? 4 : 1);
-  const int threads = C >= 128 ? 128 : ((C + 31) / 32) * 32;
-  const dim3 grid((C + threads - 1) / threads, (n_tokens + tile - 1) / tile), block(threads);
-  if (grid.y > 65535) return LLMIE_ERR_UNSUPPORTED_SIZE;
+#define LLMIE_CONV(TP, TO)                                                                                              \
+  causal_conv_launch<TP, TO>((const TP*)proj, ld, x_off, x_bias, taps, conv_bias, conv_state, cu_q, tok_seq, seq_slot,  \
+                             (TO*)u, n_tokens, C, K, act, single, stream)
+  if (dtype == LLMIE_F32 && u_dtype == LLMIE_F32) LLMIE_CONV(float, float);
+  else if (dtype == LLMIE_BF16 && u_dtype == LLMIE_F32) LLMIE_CONV(__nv_bfloat16, float);
+  else if (dtype == LLMIE_BF16 && u_dtype == LLMIE_BF16) LLMIE_CONV(__nv_bfloat16, __nv_bfloat16);
+  else if (dtype == LLMIE_F32 && u_dtype == LLMIE_BF16) LLMIE_CONV(float, __nv_bfloat16);
+  else return LLMIE_ERR_DTYPE;
+#undef LLMIE_CONV
+  LLMIE_LAUNCH_CHECK();
+  return LLMIE_OK;
+}
+
+// The state a convolution leaves behind after a step of any pieces (see conv_state_store_kernel); K >= 2.
+extern "C" int llmie_conv_state_store(const void* proj, int ld, int x_off, const float* x_bias, float* conv_state,
+                                      const int* cu_q, const int* seq_slot, int n_seqs, int C, int K, int dtype,
+                                      cudaStream_t stream) {
+  if (n_seqs < 0 || C <= 0 || K < 2 || x_off < 0 || ld < x_off + C) return LLMIE_ERR_BAD_ARG;
+  if (K > kMaxTaps || n_seqs > 65535) return LLMIE_ERR_UNSUPPORTED_SIZE;
+  if (n_seqs == 0) return LLMIE_OK;
+  const dim3 grid((C + 127) / 128, n_seqs), block(128);
   if (dtype == LLMIE_F32)
-    launch_k(causal_conv_kernel<float>, grid, block, 0, stream, (const float*)proj, ld, x_off, x_bias, taps, conv_bias,
-             conv_state, cu_q, tok_seq, seq_slot, u, C, K, n_tokens, tile);
+    launch_k(conv_state_store_kernel<float>, grid, block, 0, stream, (const float*)proj, ld, x_off, x_bias, conv_state,
+             cu_q, seq_slot, C, K);
   else if (dtype == LLMIE_BF16)
-    launch_k(causal_conv_kernel<__nv_bfloat16>, grid, block, 0, stream, (const __nv_bfloat16*)proj, ld, x_off, x_bias,
-             taps, conv_bias, conv_state, cu_q, tok_seq, seq_slot, u, C, K, n_tokens, tile);
+    launch_k(conv_state_store_kernel<__nv_bfloat16>, grid, block, 0, stream, (const __nv_bfloat16*)proj, ld, x_off, x_bias,
+             conv_state, cu_q, seq_slot, C, K);
   else
     return LLMIE_ERR_DTYPE;
   LLMIE_LAUNCH_CHECK();

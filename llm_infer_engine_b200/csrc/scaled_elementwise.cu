@@ -1,10 +1,11 @@
 // Row kernels of blocks that scale a branch's output on its way into the residual stream, and of a feed-forward whose
 // activation is a sum of normalised powers:
 //
-//   scaled_add_rmsnorm   h += s (.) (c1 d1 + c2 d2);  y = h / sqrt(mean(h^2) + eps) * w
+//   scaled_add_rmsnorm   h += s (.) (c1 d1 + c2 d2) + b;  y = h / sqrt(mean(h^2) + eps) * w
 //                        s a vector over the width (a learned scale per channel, or none), c1 and c2 constants, d1 and
-//                        d2 branch outputs (the second optional: two mixers side by side); either half may be left out:
-//                        no w and y = only the add, no d1 = only the norm
+//                        d2 branch outputs (the second optional: two mixers side by side), b a vector over the width (a
+//                        branch's output bias, or none); either half may be left out: no w and y = only the add, no d1
+//                        = only the norm, y without w = a copy of the new stream in y's type
 //   poly_norm            y = a N(z) + b N(z^2) + c N(z^3) + e, N(t) = t / sqrt(mean(t^2) + eps) over the row, powers
 //                        element by element; a, b, c, e learned numbers in device memory
 //
@@ -39,8 +40,9 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
 template <typename TY>
 __global__ void scaled_add_rmsnorm4_kernel(float* __restrict__ h, const void* __restrict__ d1, int d1_dtype, float c1,
                                            const void* __restrict__ d2, int d2_dtype, float c2,
-                                           const float* __restrict__ s, const float* __restrict__ w, float eps,
-                                           TY* __restrict__ y, const int* __restrict__ rows, int d) {
+                                           const float* __restrict__ s, const float* __restrict__ bias,
+                                           const float* __restrict__ w, float eps, TY* __restrict__ y, int y_ld,
+                                           const int* __restrict__ rows, int d) {
   extern __shared__ float row_smem[];
   __shared__ float red[32];
   pdl_launch_dependents();
@@ -63,7 +65,15 @@ __global__ void scaled_add_rmsnorm4_kernel(float* __restrict__ h, const void* __
       } else {
         x = make_float4(x.x + b.x, x.y + b.y, x.z + b.z, x.w + b.w);
       }
+      if (bias) {
+        const float4 bv = *reinterpret_cast<const float4*>(bias + c);
+        x = make_float4(x.x + bv.x, x.y + bv.y, x.z + bv.z, x.w + bv.w);
+      }
       if (!rows) *reinterpret_cast<float4*>(h + src + c) = x;
+    }
+    if (y && !w) {
+      store4(y + r_out * y_ld + c, x);
+      continue;
     }
     *reinterpret_cast<float4*>(row_smem + c) = x;
     ss = fmaf(x.x, x.x, ss);
@@ -71,21 +81,22 @@ __global__ void scaled_add_rmsnorm4_kernel(float* __restrict__ h, const void* __
     ss = fmaf(x.z, x.z, ss);
     ss = fmaf(x.w, x.w, ss);
   }
-  if (!y) return;
+  if (!y || !w) return;
   ss = block_sum(ss, red);
   const float rstd = 1.f / sqrtf(ss / (float)d + eps);
   for (int c = threadIdx.x * 4; c < d; c += blockDim.x * 4) {
     const float4 x = *reinterpret_cast<const float4*>(row_smem + c);
     const float4 wv = *reinterpret_cast<const float4*>(w + c);
-    store4(y + r_out * d + c, make_float4(x.x * rstd * wv.x, x.y * rstd * wv.y, x.z * rstd * wv.z, x.w * rstd * wv.w));
+    store4(y + r_out * y_ld + c, make_float4(x.x * rstd * wv.x, x.y * rstd * wv.y, x.z * rstd * wv.z, x.w * rstd * wv.w));
   }
 }
 
 template <typename TY>
 __global__ void scaled_add_rmsnorm_kernel(float* __restrict__ h, const void* __restrict__ d1, int d1_dtype, float c1,
                                           const void* __restrict__ d2, int d2_dtype, float c2,
-                                          const float* __restrict__ s, const float* __restrict__ w, float eps,
-                                          TY* __restrict__ y, const int* __restrict__ rows, int d) {
+                                          const float* __restrict__ s, const float* __restrict__ bias,
+                                          const float* __restrict__ w, float eps, TY* __restrict__ y, int y_ld,
+                                          const int* __restrict__ rows, int d) {
   extern __shared__ float row_smem[];
   __shared__ float red[32];
   pdl_launch_dependents();
@@ -99,15 +110,20 @@ __global__ void scaled_add_rmsnorm_kernel(float* __restrict__ h, const void* __r
       float b = c1 * load_any(d1, d1_dtype, src + c);
       if (d2) b = fmaf(c2, load_any(d2, d2_dtype, src + c), b);
       x = s ? fmaf(s[c], b, x) : x + b;
+      if (bias) x += bias[c];
       if (!rows) h[src + c] = x;
+    }
+    if (y && !w) {
+      y[r_out * y_ld + c] = from_f32<TY>(x);
+      continue;
     }
     row_smem[c] = x;
     ss = fmaf(x, x, ss);
   }
-  if (!y) return;
+  if (!y || !w) return;
   ss = block_sum(ss, red);
   const float rstd = 1.f / sqrtf(ss / (float)d + eps);
-  for (int c = threadIdx.x; c < d; c += blockDim.x) y[r_out * d + c] = from_f32<TY>(row_smem[c] * rstd * w[c]);
+  for (int c = threadIdx.x; c < d; c += blockDim.x) y[r_out * y_ld + c] = from_f32<TY>(row_smem[c] * rstd * w[c]);
 }
 
 template <typename T>
@@ -190,13 +206,15 @@ static inline int row_block(int d) {
 
 using namespace llmie;
 
-// h float32 [T, d]; d1, d2 (d2 only with d1) [T, d] of their own dtypes, or null; s float32 [d] or null; w float32 [d]
-// with y [n_out, d] of y_dtype, or both null (the add alone); rows int32 [n_out] or null (then n_out == T and h is
-// updated in place). A row must fit shared memory (d <= 12,288).
+// h float32 [T, d]; d1, d2 (d2 only with d1) [T, d] of their own dtypes, or null; s, bias float32 [d] or null (bias only
+// with d1); y rows of d elements of y_dtype, y_ld apart, or null (the add alone); w float32 [d] or null (with y: the new
+// stream itself is stored); rows int32 [n_out] or null (then n_out == T and h is updated in place). A row must fit shared
+// memory (d <= 12,288).
 extern "C" int llmie_scaled_add_rmsnorm(float* h, const void* d1, int d1_dtype, float c1, const void* d2, int d2_dtype,
-                                        float c2, const float* s, const float* w, float eps, void* y, int y_dtype,
-                                        const int* rows, int n_out, int d, cudaStream_t stream) {
-  if (n_out < 0 || d <= 0 || !h || (d2 && !d1) || (!y) != (!w) || (!y && (rows || !d1))) return LLMIE_ERR_BAD_ARG;
+                                        float c2, const float* s, const float* bias, const float* w, float eps, void* y,
+                                        int y_ld, int y_dtype, const int* rows, int n_out, int d, cudaStream_t stream) {
+  if (n_out < 0 || d <= 0 || !h || (d2 && !d1) || (bias && !d1) || (w && !y) || (!y && (rows || !d1)) || (y && y_ld < d))
+    return LLMIE_ERR_BAD_ARG;
   if ((y && y_dtype != LLMIE_F32 && y_dtype != LLMIE_BF16) || (d1 && d1_dtype != LLMIE_F32 && d1_dtype != LLMIE_BF16) ||
       (d2 && d2_dtype != LLMIE_F32 && d2_dtype != LLMIE_BF16))
     return LLMIE_ERR_DTYPE;
@@ -204,24 +222,24 @@ extern "C" int llmie_scaled_add_rmsnorm(float* h, const void* d1, int d1_dtype, 
   if (n_out == 0) return LLMIE_OK;
   const dim3 grid(n_out), block(row_block(d));
   const size_t smem = (size_t)d * sizeof(float);
-  const bool by4 = d % 4 == 0 && aligned16(h) && (!s || aligned16(s)) && (!w || aligned16(w)) &&
-                   (!d1 || aligned16(d1)) && (!d2 || aligned16(d2)) && (!y || aligned16(y));
+  const bool by4 = d % 4 == 0 && aligned16(h) && (!s || aligned16(s)) && (!w || aligned16(w)) && (!bias || aligned16(bias)) &&
+                   (!d1 || aligned16(d1)) && (!d2 || aligned16(d2)) && (!y || (aligned16(y) && y_ld % 4 == 0));
   if (by4) {
     if (y && y_dtype == LLMIE_BF16)
       launch_k(scaled_add_rmsnorm4_kernel<__nv_bfloat16>, grid, block, smem, stream, h, d1, d1_dtype, c1, d2, d2_dtype,
-               c2, s, w, eps, (__nv_bfloat16*)y, rows, d);
+               c2, s, bias, w, eps, (__nv_bfloat16*)y, y_ld, rows, d);
     else
-      launch_k(scaled_add_rmsnorm4_kernel<float>, grid, block, smem, stream, h, d1, d1_dtype, c1, d2, d2_dtype, c2, s, w,
-               eps, (float*)y, rows, d);
+      launch_k(scaled_add_rmsnorm4_kernel<float>, grid, block, smem, stream, h, d1, d1_dtype, c1, d2, d2_dtype, c2, s,
+               bias, w, eps, (float*)y, y_ld, rows, d);
     LLMIE_LAUNCH_CHECK();
     return LLMIE_OK;
   }
   if (y && y_dtype == LLMIE_BF16)
     launch_k(scaled_add_rmsnorm_kernel<__nv_bfloat16>, grid, block, smem, stream, h, d1, d1_dtype, c1, d2, d2_dtype, c2, s,
-             w, eps, (__nv_bfloat16*)y, rows, d);
+             bias, w, eps, (__nv_bfloat16*)y, y_ld, rows, d);
   else
-    launch_k(scaled_add_rmsnorm_kernel<float>, grid, block, smem, stream, h, d1, d1_dtype, c1, d2, d2_dtype, c2, s, w,
-             eps, (float*)y, rows, d);
+    launch_k(scaled_add_rmsnorm_kernel<float>, grid, block, smem, stream, h, d1, d1_dtype, c1, d2, d2_dtype, c2, s, bias, w,
+             eps, (float*)y, y_ld, rows, d);
   LLMIE_LAUNCH_CHECK();
   return LLMIE_OK;
 }

@@ -50,7 +50,7 @@ class KernelPlan:
         n_runs = ((ctx.max_kv_len + 63) // 64 + pages - 1) // pages
         counters = self._decode_counters(ops.decode_counter_ints(ctx.n_seqs, n_q, n_kv), qkv.device)
         ops.attention_decode_mma_rope(qkv, kv.k, kv.v, out, table, ctx.seq_slot, ctx.seq_kvlen, kv.block_table,
-                                      kv.page_size, n_q, n_kv, head_dim, options.scale, options.window, pages, n_runs,
+                                      kv.page_size, n_q, n_kv, head_dim, options.scale, options.reach, pages, n_runs,
                                       write_kv, counters=counters)
         return True
 
@@ -58,7 +58,7 @@ class KernelPlan:
         """Returns True when a specialised kernel ran (the gate, if any, applied). The tensor-core kernels know
         every option (scale, window, kept first keys, sink, gate); the CUDA-core split-KV kernel knows scale and
         window. A value head size that differs from the key head size is the plain kernel's alone."""
-        scale, window = options.scale, options.window
+        scale, window = options.scale, options.reach
         if options.sigmoid_bias is not None:
             return self._sigmoid_attention(ctx, q, kv, out, n_q, n_kv, head_dim, options, gate)
         if kv.v.shape[-1] != head_dim or not kv.v.is_contiguous():
@@ -101,7 +101,8 @@ class KernelPlan:
             if gate is not None:
                 ops.sigmoid_gate(out, gate)
             return True
-        return False
+        # head sizes that none of the kernels above takes
+        return self._attention_by_rows(ctx, q, kv, out, n_q, n_kv, head_dim, options, gate)
 
     def _sigmoid_attention(self, ctx, q, kv, out, n_q, n_kv, head_dim, options, gate) -> bool:
         """Attention without a softmax (weights sigmoid(score + a number per head), not normalised). Prompts of the
@@ -114,7 +115,7 @@ class KernelPlan:
                 and ops.attention_prefill_tc_supported(head_dim, kv.page_size, q.dtype):
             ops.attention_prefill_tc(q, kv.k, kv.v, out, ctx.cu_q, ctx.seq_slot, ctx.seq_start, kv.block_table,
                                      kv.page_size, ctx.n_seqs, ctx.max_q_len, n_q, n_kv, head_dim, options.scale,
-                                     options.window, options.keep_first, False, gate,
+                                     options.reach, options.keep_first, False, gate,
                                      sigmoid_bias=options.sigmoid_bias)
             return True
         if ctx.decode and self.decode_attention != "split" and square and aligned_gate \
@@ -123,7 +124,7 @@ class KernelPlan:
             n_runs = ((ctx.max_kv_len + 63) // 64 + pages - 1) // pages
             counters = self._decode_counters(ops.decode_counter_ints(ctx.n_seqs, n_q, n_kv), q.device)
             ops.attention_decode_mma(q, kv.k, kv.v, out, ctx.seq_slot, ctx.seq_kvlen, kv.block_table, kv.page_size,
-                                     n_q, n_kv, head_dim, options.scale, options.window, pages, n_runs,
+                                     n_q, n_kv, head_dim, options.scale, options.reach, pages, n_runs,
                                      counters=counters, keep_first=options.keep_first, gate=gate,
                                      sigmoid_bias=options.sigmoid_bias)
             return True
@@ -137,7 +138,7 @@ class KernelPlan:
                                                                       shared_rows):
             return False
         ops.attention_rows_mma(q, kv.k, kv.v, out, ctx.cu_q, ctx.seq_slot, ctx.seq_start, kv.block_table, kv.page_size,
-                               ctx.n_seqs, ctx.max_q_len, n_q, n_kv, head_dim, options.scale, options.window,
+                               ctx.n_seqs, ctx.max_q_len, n_q, n_kv, head_dim, options.scale, options.reach,
                                options.softcap, options.distance_bias, options.sink_values, options.sink,
                                options.sigmoid_bias)
         if gate is not None:

@@ -33,6 +33,8 @@ FAMILIES: Dict[str, tuple] = {
     "parallel_elementwise": ("parallel_elementwise.cu", [], []),
     "scaled_elementwise": ("scaled_elementwise.cu", [], []),
     "recurrent": ("recurrent.cu", [], []),
+    "ssm": ("ssm.cu", [], []),
+    "conv_attention": ("conv_attention.cu", [], []),
     "grouped_gemm": ("grouped_gemm.cu", [], []),
     "moe": ("moe.cu", [], []),
     "latent": ("latent.cu", [], []),

@@ -261,7 +261,8 @@ def attention_paged(q, k_cache, v_cache, out, tok_pos, tok_seq, seq_slot, block_
                     sigmoid_bias: Optional[torch.Tensor] = None):
     """Plain attention over the paged cache, one warp per (token, query head).
     q [T, n_q hd]; out [T, n_q hdv]; k_cache [n_pages, n_kv, page_size, hd]; v_cache the same with hdv (the value
-    head size, read from its shape). window 0 = all earlier keys; the first `keep_first` keys of a sequence stay
+    head size, read from its shape). window 0 = all earlier keys, n > 0 = the last n, -n < 0 = the token's own chunk of n
+    positions (every attention kernel here takes it so); the first `keep_first` keys of a sequence stay
     visible behind the window; `sink` adds a key of score 0 without a value to the softmax; `gate` (rows of
     n_q hdv elements, possibly a column slice of a wider tensor) multiplies the output by its sigmoid. `softcap` c > 0
     turns a scaled score s into c tanh(s / c); `dist_bias` (float32 [n_q, L]) adds a number per head and distance
@@ -754,6 +755,22 @@ def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: i
     _work(_nbytes(x, w, out), 2.0 * x.shape[0] * w.shape[0] * w.shape[1])
     f = _fn("gemm_skinny", "llmie_gemm_skinny", [_c_void_p] * 3 + [_c_int] * 5 + [_c_void_p])
     _check(f(x.data_ptr(), w.data_ptr(), out.data_ptr(), batch, N, K, cols, epilogue, _stream()), "gemm_skinny")
+    return out
+
+
+def gemm_skinny_add_bias(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: torch.Tensor) -> torch.Tensor:
+    """out (float32 [batch, N]) += x w^T + bias (float32 [N]): gemm_skinny's add with a bias."""
+    batch, K = x.shape
+    N = w.shape[0]
+    _need(x, "x", torch.bfloat16)
+    _need(w, "w", torch.bfloat16, (N, K))
+    _need(out, "out", torch.float32, (batch, N))
+    _need(bias, "bias", torch.float32, (N,))
+    if not gemm_skinny_ok(batch, N, K):
+        raise KernelError(f"gemm_skinny_add_bias: shape batch={batch}, N={N}, K={K} is not supported")
+    _work(_nbytes(x, w, out), 2.0 * batch * N * K)
+    f = _fn("gemm_skinny", "llmie_gemm_skinny_add_bias", [_c_void_p] * 3 + [_c_int] * 4 + [_c_void_p, _c_void_p])
+    _check(f(x.data_ptr(), w.data_ptr(), out.data_ptr(), batch, N, K, N, bias.data_ptr(), _stream()), "gemm_skinny_add")
     return out
 
 
@@ -1564,11 +1581,15 @@ def attention_rows_mma(q, k_cache, v_cache, out, cu_q, seq_slot, seq_start, bloc
 
 
 # ------------------------------------------------------------------------------------------ scaled branches, PolyNorm
-def scaled_add_rmsnorm(h, d1, c1: float, d2, c2: float, scale, weight, eps: float, out, rows=None):
-    """h += scale (.) (c1 d1 + c2 d2) (float32, in place, when rows is None); out = rmsnorm(h) * weight.
-    h float32 [T, d]; d1, d2 [T, d] float32 or bfloat16 (d2 or both may be None); scale float32 [d] or None; weight
-    float32 [d] with out [n_out, d], or both None (the add alone). With `rows` (int32 [n_out]) only those rows are
-    produced and h stays as it is."""
+SCALED_ADD_MAX_WIDTH = 12288     # a row in shared memory
+
+
+def scaled_add_rmsnorm(h, d1, c1: float, d2, c2: float, scale, weight, eps: float, out, rows=None, bias=None):
+    """h += scale (.) (c1 d1 + c2 d2) + bias (float32, in place, when rows is None); out = rmsnorm(h) * weight.
+    h float32 [T, d]; d1, d2 [T, d] float32 or bfloat16 (d2 or both may be None); scale, bias float32 [d] or None (bias
+    only with d1); weight float32 [d] with out [n_out, d] (possibly a column slice), or both None (the add alone), or only
+    out (the new stream itself, in out's type). With `rows` (int32 [n_out]) only those rows are produced and h stays as it
+    is."""
     T, d = h.shape
     n_out = T if rows is None else rows.shape[0]
     _need(h, "h", torch.float32)
@@ -1577,22 +1598,26 @@ def scaled_add_rmsnorm(h, d1, c1: float, d2, c2: float, scale, weight, eps: floa
             _need(t, name, None, (T, d))
     if scale is not None:
         _need(scale, "scale", torch.float32, (d,))
-    if (weight is None) != (out is None):
-        raise KernelError("scaled_add_rmsnorm: weight and out go together")
-    if out is not None:
+    if weight is not None and out is None:
+        raise KernelError("scaled_add_rmsnorm: a weight needs an out")
+    if bias is not None:
+        _need(bias, "bias", torch.float32, (d,))
+        if d1 is None:
+            raise KernelError("scaled_add_rmsnorm: a bias needs a branch output")
+    if weight is not None:
         _need(weight, "weight", torch.float32, (d,))
-        _need(out, "out", None, (n_out, d))
     if rows is not None:
         _need(rows, "rows", torch.int32, (n_out,))
         if n_out == 0:
             return out                   # no row is wanted and h stays as it is
+    out_ld = _row_slice(out, "out", out.dtype, n_out, d) if out is not None else d
     _work((2 * _nbytes(h) if rows is None else n_out * d * 4) + _nbytes(d1, d2, out))
     f = _fn("scaled_elementwise", "llmie_scaled_add_rmsnorm",
-            [_c_void_p, _c_void_p, _c_int, _c_float, _c_void_p, _c_int, _c_float, _c_void_p, _c_void_p, _c_float,
-             _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p])
+            [_c_void_p, _c_void_p, _c_int, _c_float, _c_void_p, _c_int, _c_float, _c_void_p, _c_void_p, _c_void_p,
+             _c_float, _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_void_p])
     _check(f(h.data_ptr(), _ptr(d1), _dt(d1, "d1") if d1 is not None else 0, float(c1), _ptr(d2),
-             _dt(d2, "d2") if d2 is not None else 0, float(c2), _ptr(scale), _ptr(weight), float(eps), _ptr(out),
-             _dt(out, "out") if out is not None else 0, _ptr(rows), n_out, d, _stream()), "scaled_add_rmsnorm")
+             _dt(d2, "d2") if d2 is not None else 0, float(c2), _ptr(scale), _ptr(bias), _ptr(weight), float(eps),
+             _ptr(out), int(out_ld), _dt(out, "out") if out is not None else 0, _ptr(rows), n_out, d, _stream()), "scaled_add_rmsnorm")
     return out
 
 
@@ -1639,19 +1664,30 @@ SCAN_SCRATCH_BYTES = 1 << 30
 
 
 def matrix_scan(q, f, v, state, cu_q, seq_slot, out, n_seqs: int, heads: int, dim: int, vdim: int,
-                write_state: bool = True, max_len: int = 0, head_decay: Optional[torch.Tensor] = None):
+                write_state: bool = True, max_len: int = 0, head_decay: Optional[torch.Tensor] = None,
+                key_factor: Optional[torch.Tensor] = None, groups: Optional[int] = None):
     """Per sequence and head, from the state S [dim, vdim] the slot holds: S <- diag(f_t) S + (1 - f_t) v_t^T and
     out_t = S^T q_t for each of the step's tokens in order; the new S is written back. q, f float32 [T, heads dim];
     v [T, heads vdim] (possibly a column slice) float32 or bfloat16; state float32 [slots, heads, dim, vdim];
     out float32 [T, heads vdim]. `max_len`: an upper bound of the longest piece, if the caller knows one; long pieces
     are cut into chunks that run side by side (each chunk from zero, a chain over the chunks' ends, each chunk again
     from its true start), which changes rounding only. With `head_decay` (float32 [heads]) the recurrence is the
-    keyed one, S <- head_decay[h] S + k_t v_t^T, and `f` holds the keys k (linear attention with a constant decay)."""
+    keyed one, S <- head_decay[h] S + k_t v_t^T, and `f` holds the keys k (linear attention with a constant decay). With
+    `key_factor` as well (both float32 [T, heads] then) it is the stepped one, S <- head_decay[t, h] S +
+    (key_factor[t, h] k_t) v_t^T, and q and f have `groups` heads, each shared by heads / groups heads of the state."""
     T = q.shape[0]
-    if head_decay is not None:
+    stepped = key_factor is not None
+    n_qk = heads
+    if stepped:
+        n_qk = heads if groups is None else int(groups)
+        if n_qk <= 0 or heads % n_qk:
+            raise KernelError(f"matrix_scan: {heads} heads are not whole groups of {n_qk}")
+        _need(head_decay, "head_decay", torch.float32, (T, heads))
+        _need(key_factor, "key_factor", torch.float32, (T, heads))
+    elif head_decay is not None:
         _need(head_decay, "head_decay", torch.float32, (heads,))
-    _need(q, "q", torch.float32, (T, heads * dim))
-    _need(f, "f", torch.float32, (T, heads * dim))
+    _need(q, "q", torch.float32, (T, n_qk * dim))
+    _need(f, "f", torch.float32, (T, n_qk * dim))
     _need(state, "state", torch.float32, (None, heads, dim, vdim))
     _need(out, "out", torch.float32, (T, heads * vdim))
     _need(cu_q, "cu_q", torch.int32)
@@ -1668,6 +1704,10 @@ def matrix_scan(q, f, v, state, cu_q, seq_slot, out, n_seqs: int, heads: int, di
             ws = torch.empty((n_seqs, n_chunks, heads, dim, vdim), dtype=torch.float32, device=q.device)
             decay = torch.empty((n_seqs, n_chunks, heads, dim), dtype=torch.float32, device=q.device)
             _work(3.0 * _nbytes(ws) + _nbytes(f) + T * heads * vdim * v.element_size(), 4.0 * T * heads * dim * vdim)
+            if stepped:
+                _matrix_scan_stepped(q, f, v, v_ld, state, cu_q, seq_slot, out, ws, decay, n_seqs, heads, n_qk, dim, vdim,
+                                     chunk, n_chunks, write_state, head_decay, key_factor)
+                return out
             f_ = _fn("recurrent", "llmie_matrix_scan_chunked_ex",
                      [_c_void_p, _c_void_p, _c_void_p, _c_int] + [_c_void_p] * 6 + [_c_int] * 8 + [_c_void_p, _c_void_p])
             _check(f_(q.data_ptr(), f.data_ptr(), v.data_ptr(), v_ld, state.data_ptr(), cu_q.data_ptr(),
@@ -1675,12 +1715,26 @@ def matrix_scan(q, f, v, state, cu_q, seq_slot, out, n_seqs: int, heads: int, di
                       chunk, n_chunks, 1 if write_state else 0, _dt(v, "v"), _ptr(head_decay), _stream()),
                    "matrix_scan_chunked")
             return out
+    if stepped:
+        _matrix_scan_stepped(q, f, v, v_ld, state, cu_q, seq_slot, out, None, None, n_seqs, heads, n_qk, dim, vdim, 0, 1,
+                             write_state, head_decay, key_factor)
+        return out
     f_ = _fn("recurrent", "llmie_matrix_scan_ex", [_c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p,
                                                    _c_void_p, _c_void_p] + [_c_int] * 6 + [_c_void_p, _c_void_p])
     _check(f_(q.data_ptr(), f.data_ptr(), v.data_ptr(), v_ld, state.data_ptr(), cu_q.data_ptr(), seq_slot.data_ptr(),
               out.data_ptr(), n_seqs, heads, dim, vdim, 1 if write_state else 0, _dt(v, "v"), _ptr(head_decay),
               _stream()), "matrix_scan")
     return out
+
+
+def _matrix_scan_stepped(q, f, v, v_ld, state, cu_q, seq_slot, out, ws, decay, n_seqs, heads, groups, dim, vdim, chunk,
+                         n_chunks, write_state, token_decay, key_factor):
+    f_ = _fn("recurrent", "llmie_matrix_scan_stepped",
+             [_c_void_p, _c_void_p, _c_void_p, _c_int] + [_c_void_p] * 6 + [_c_int] * 9 + [_c_void_p] * 3)
+    _check(f_(q.data_ptr(), f.data_ptr(), v.data_ptr(), v_ld, state.data_ptr(), cu_q.data_ptr(), seq_slot.data_ptr(),
+              out.data_ptr(), _ptr(ws), _ptr(decay), n_seqs, heads, groups, dim, vdim, chunk, n_chunks,
+              1 if write_state else 0, _dt(v, "v"), token_decay.data_ptr(), key_factor.data_ptr(), _stream()),
+           "matrix_scan_stepped")
 
 
 def head_rmsnorm(o, weight, eps: float, out, vdim: int, gate=None):
@@ -1724,26 +1778,185 @@ def act_columns(proj, runs, act: int):
     _check(f(proj.data_ptr(), ld, *args, int(act), T, _dt(proj, "proj"), _stream()), "act_columns")
 
 
-def causal_conv(proj, x_off: int, x_bias, taps, conv_bias, conv_state, cu_q, tok_seq, seq_slot, out):
-    """out[t, c] = conv_bias[c] + sum_j taps[c, K-1-j] x[t-j, c] with x = proj[:, x_off + c] + x_bias[c]; inputs from
+def causal_conv(proj, x_off: int, x_bias, taps, conv_bias, conv_state, cu_q, tok_seq, seq_slot, out, act: int = ACT_NONE,
+                single: bool = False):
+    """out[t, c] = act(conv_bias[c] + sum_j taps[c, K-1-j] x[t-j, c]) with x = proj[:, x_off + c] + x_bias[c]; inputs from
     before the step are the slot's conv_state (its last K-1 inputs, zeros at a sequence's start).
-    taps float32 [C, K]; conv_state float32 [slots, K-1, C]; out float32 [T, C]."""
+    taps float32 [C, K]; conv_state float32 [slots, K-1, C] (None with K = 1); out [T, C] float32 or bfloat16. `single`:
+    every sequence of the step brings one token, and the new conv_state is written too (`conv_state_store` does it for
+    other steps)."""
     T, C = out.shape
     K = taps.shape[1]
     _need(proj, "proj", None, (T, None))
     _need(taps, "taps", torch.float32, (C, K))
-    _need(conv_state, "conv_state", torch.float32, (None, K - 1, C))
-    _need(out, "out", torch.float32)
+    if K > 1:
+        _need(conv_state, "conv_state", torch.float32, (None, K - 1, C))
+    _need(out, "out")
     for name, t in (("x_bias", x_bias), ("conv_bias", conv_bias)):
         if t is not None:
             _need(t, name, torch.float32, (C,))
     for name, t in (("cu_q", cu_q), ("tok_seq", tok_seq), ("seq_slot", seq_slot)):
         _need(t, name, torch.int32)
-    _work(T * C * (proj.element_size() + 4))
-    f = _fn("recurrent", "llmie_causal_conv", [_c_void_p, _c_int, _c_int] + [_c_void_p] * 8 + [_c_int] * 4 + [_c_void_p])
+    _work(T * C * (proj.element_size() + out.element_size()))
+    f = _fn("recurrent", "llmie_causal_conv_ex",
+            [_c_void_p, _c_int, _c_int] + [_c_void_p] * 8 + [_c_int] * 7 + [_c_void_p])
     _check(f(proj.data_ptr(), proj.shape[1], int(x_off), _ptr(x_bias), taps.data_ptr(), _ptr(conv_bias),
-             conv_state.data_ptr(), cu_q.data_ptr(), tok_seq.data_ptr(), seq_slot.data_ptr(), out.data_ptr(), T, C, K,
-             _dt(proj, "proj"), _stream()), "causal_conv")
+             _ptr(conv_state), cu_q.data_ptr(), tok_seq.data_ptr(), seq_slot.data_ptr(), out.data_ptr(), _dt(out, "out"),
+             T, C, K, int(act), 1 if single and K > 1 else 0, _dt(proj, "proj"), _stream()), "causal_conv")
+    return out
+
+
+def conv_state_store(proj, x_off: int, x_bias, conv_state, cu_q, seq_slot, n_seqs: int):
+    """Leaves the last K-1 inputs x = proj[:, x_off + c] + x_bias[c] of every sequence of the step in its slot's conv_state
+    (float32 [slots, K-1, C]); inputs from before the step move up."""
+    _need(proj, "proj")
+    _need(conv_state, "conv_state", torch.float32, (None, None, None))
+    K, C = conv_state.shape[1] + 1, conv_state.shape[2]
+    if x_bias is not None:
+        _need(x_bias, "x_bias", torch.float32, (C,))
+    _need(cu_q, "cu_q", torch.int32)
+    _need(seq_slot, "seq_slot", torch.int32)
+    f = _fn("recurrent", "llmie_conv_state_store",
+            [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p] + [_c_int] * 4 + [_c_void_p])
+    _check(f(proj.data_ptr(), proj.shape[1], int(x_off), _ptr(x_bias), conv_state.data_ptr(), cu_q.data_ptr(),
+             seq_slot.data_ptr(), n_seqs, C, K, _dt(proj, "proj"), _stream()), "conv_state_store")
+
+
+def conv_qk_store(proj, bias, taps, conv_state, q_w, k_w, eps: float, table, rot_dim: int, cu_q, tok_pos, tok_seq, seq_slot,
+                  block_table, page_size: int, q_out, k_cache, v_cache, n_q: int, n_kv: int, head_dim: int,
+                  single: bool = False):
+    """What stands between the q and k projections of a layer with a short convolution and its attention: bias, a causal
+    convolution per channel over time, RMS norm per head, rotation of the first rot_dim channels in pairs (2i, 2i + 1), and
+    the cache write; the stored values are the keys as the convolution leaves them. proj [T, >= C] holds the q heads and
+    then the k heads (C = (n_q + n_kv) head_dim), float32 or bfloat16; bias float32 [C] or None; taps float32 [C, K];
+    conv_state float32 [slots, K-1, C] (None with K = 1); q_w, k_w float32 [head_dim]; table float32 [positions,
+    rot_dim / 2, 2] of (cos, sin); q_out [T, n_q head_dim] and the caches of one dtype. `single`: every sequence brings one
+    token, and the new conv_state is written too (`conv_state_store` does it for other steps)."""
+    T, ld = proj.shape
+    C, K = (n_q + n_kv) * head_dim, taps.shape[1]
+    _need(proj, "proj")
+    if ld < C:
+        raise KernelError(f"conv_qk_store: rows of {ld} elements cannot hold q and k ({C})")
+    _need(taps, "taps", torch.float32, (C, K))
+    if bias is not None:
+        _need(bias, "bias", torch.float32, (C,))
+    if K > 1:
+        _need(conv_state, "conv_state", torch.float32, (None, K - 1, C))
+    _need(q_w, "q_w", torch.float32, (head_dim,))
+    _need(k_w, "k_w", torch.float32, (head_dim,))
+    _need(table, "table", torch.float32, (None, rot_dim // 2, 2))
+    for name, t in (("cu_q", cu_q), ("tok_pos", tok_pos), ("tok_seq", tok_seq), ("seq_slot", seq_slot),
+                    ("block_table", block_table)):
+        _need(t, name, torch.int32)
+    _need(q_out, "q_out", None, (T, n_q * head_dim))
+    _need(k_cache, "k_cache", q_out.dtype, (None, n_kv, page_size, head_dim))
+    _need(v_cache, "v_cache", q_out.dtype, tuple(k_cache.shape))
+    _work(T * C * proj.element_size() + _nbytes(q_out) + 2 * T * n_kv * head_dim * q_out.element_size())
+    f = _fn("conv_attention", "llmie_conv_qk_store",
+            [_c_void_p, _c_int] + [_c_void_p] * 5 + [_c_float, _c_void_p, _c_int, _c_int] + [_c_void_p] * 5 +
+            [_c_int, _c_int] + [_c_void_p] * 3 + [_c_int] * 8 + [_c_void_p])
+    _check(f(proj.data_ptr(), ld, _ptr(bias), taps.data_ptr(), _ptr(conv_state), q_w.data_ptr(), k_w.data_ptr(), float(eps),
+             table.data_ptr(), table.shape[0], int(rot_dim), cu_q.data_ptr(), tok_pos.data_ptr(), tok_seq.data_ptr(),
+             seq_slot.data_ptr(), block_table.data_ptr(), block_table.shape[1], page_size, q_out.data_ptr(),
+             k_cache.data_ptr(), v_cache.data_ptr(), T, n_q, n_kv, head_dim, K, 1 if single and K > 1 else 0,
+             _dt(proj, "proj"), _dt(q_out, "q_out"), _stream()), "conv_qk_store")
+    return q_out
+
+
+# ------------------------------------------------------------------------------------------ state space layers
+def ssm_scan_supported(state: int, vdim: int) -> bool:
+    """The sizes ssm_scan takes (answered without loading the library)."""
+    return state % 8 == 0 and vdim % 8 == 0 and 0 < state <= 256 and vdim > 0
+
+
+def ssm_steps(proj, dt_off: int, dt_bias, A, dt, decay):
+    """dt = softplus(proj[:, dt_off : dt_off + H] + dt_bias), decay = exp(-A dt); dt_bias, A float32 [H]; dt, decay float32
+    [T, H]."""
+    T, H = dt.shape
+    _need(proj, "proj", None, (T, None))
+    _need(dt_bias, "dt_bias", torch.float32, (H,))
+    _need(A, "A", torch.float32, (H,))
+    _need(dt, "dt", torch.float32)
+    _need(decay, "decay", torch.float32, (T, H))
+    _work(T * H * (proj.element_size() + 8))
+    f = _fn("ssm", "llmie_ssm_steps", [_c_void_p, _c_int, _c_int] + [_c_void_p] * 4 + [_c_int] * 3 + [_c_void_p])
+    _check(f(proj.data_ptr(), proj.shape[1], int(dt_off), dt_bias.data_ptr(), A.data_ptr(), dt.data_ptr(),
+             decay.data_ptr(), T, H, _dt(proj, "proj"), _stream()), "ssm_steps")
+
+
+def _ssm_common(what, proj, dt_off, dt_bias, A, skip, xbc, xbc_dtype, state, cu_q, seq_slot, out, heads, groups, dim, vdim):
+    T = proj.shape[0]
+    _need(proj, "proj")
+    for name, t in (("dt_bias", dt_bias), ("A", A), ("skip", skip)):
+        _need(t, name, torch.float32, (heads,))
+    if groups <= 0 or heads % groups:
+        raise KernelError(f"{what}: {heads} heads are not whole groups of {groups}")
+    _need(xbc, "xbc", xbc_dtype, (T, heads * vdim + 2 * groups * dim))
+    _need(state, "state", torch.float32, (None, heads, dim, vdim))
+    _need(out, "out", torch.float32, (T, heads * vdim))
+    _need(cu_q, "cu_q", torch.int32)
+    _need(seq_slot, "seq_slot", torch.int32)
+
+
+def ssm_step(proj, dt_off: int, dt_bias, A, skip, xbc, state, cu_q, seq_slot, out, n_seqs: int, heads: int, groups: int,
+             dim: int, vdim: int, write_state: bool = True):
+    """One token a sequence of S <- exp(-A dt) S + dt B x^T, out = S^T C + skip x, dt = softplus(raw + dt_bias) with raw =
+    proj[:, dt_off + h]. xbc float32 [T, H P + 2 G N] = [x | B | C]; state float32 [slots, H, N, P], updated in place; dt_bias,
+    A, skip float32 [H]; out float32 [T, H P]."""
+    _ssm_common("ssm_step", proj, dt_off, dt_bias, A, skip, xbc, torch.float32, state, cu_q, seq_slot, out, heads, groups,
+                dim, vdim)
+    _work(_nbytes(xbc, out) + (2.0 if write_state else 1.0) * n_seqs * heads * dim * vdim * 4,
+          6.0 * n_seqs * heads * dim * vdim)
+    f = _fn("ssm", "llmie_ssm_step", [_c_void_p, _c_int, _c_int] + [_c_void_p] * 4 + [_c_int] + [_c_void_p] * 4 +
+            [_c_int] * 7 + [_c_void_p])
+    _check(f(proj.data_ptr(), proj.shape[1], int(dt_off), dt_bias.data_ptr(), A.data_ptr(), skip.data_ptr(),
+             xbc.data_ptr(), xbc.shape[1], state.data_ptr(), cu_q.data_ptr(), seq_slot.data_ptr(), out.data_ptr(), n_seqs,
+             heads, groups, dim, vdim, 1 if write_state else 0, _dt(proj, "proj"), _stream()), "ssm_step")
+    return out
+
+
+def ssm_scan(proj, dt_off: int, dt_bias, A, skip, xbc, state, cu_q, seq_slot, out, n_seqs: int, heads: int, groups: int,
+             dim: int, vdim: int, write_state: bool = True):
+    """ssm_step's recurrence over pieces of any length on the tensor cores, 64 tokens at a time; xbc bfloat16. Sizes:
+    `ssm_scan_supported`."""
+    _ssm_common("ssm_scan", proj, dt_off, dt_bias, A, skip, xbc, torch.bfloat16, state, cu_q, seq_slot, out, heads, groups,
+                dim, vdim)
+    if not ssm_scan_supported(dim, vdim):
+        raise KernelError(f"ssm_scan: a state of {dim} x {vdim} is not supported")
+    T = proj.shape[0]
+    _work(_nbytes(xbc, out) + 2.0 * n_seqs * heads * dim * vdim * 4, T * heads * (4.0 * dim * vdim + 64.0 * (dim + vdim)))
+    f = _fn("ssm", "llmie_ssm_scan", [_c_void_p, _c_int, _c_int] + [_c_void_p] * 4 + [_c_int] + [_c_void_p] * 4 +
+            [_c_int] * 7 + [_c_void_p])
+    _check(f(proj.data_ptr(), proj.shape[1], int(dt_off), dt_bias.data_ptr(), A.data_ptr(), skip.data_ptr(),
+             xbc.data_ptr(), xbc.shape[1], state.data_ptr(), cu_q.data_ptr(), seq_slot.data_ptr(), out.data_ptr(), n_seqs,
+             heads, groups, dim, vdim, 1 if write_state else 0, _dt(proj, "proj"), _stream()), "ssm_scan")
+    return out
+
+
+def gated_group_norm(y, z, weight, eps: float, out, groups: int, skip_x=None, skip=None):
+    """out = v / sqrt(mean(v^2) + eps) * weight over each of `groups` equal runs of columns, v = y silu(z). y float32 [T, n];
+    z [T, n] possibly a column slice; weight float32 [n]; out [T, n]. With `skip_x` (float32 [T, n], possibly a column slice)
+    and `skip` (float32 [heads]) y + skip[head] skip_x takes the place of y."""
+    T, n = y.shape
+    _need(y, "y", torch.float32)
+    _need(weight, "weight", torch.float32, (n,))
+    _need(out, "out", None, (T, n))
+    if groups <= 0 or n % groups:
+        raise KernelError(f"gated_group_norm: {n} columns are not {groups} equal runs")
+    z_ld = _row_slice(z, "z", z.dtype, T, n)
+    x_ld, width = 0, 1
+    if skip is not None:
+        _need(skip, "skip", torch.float32)
+        if n % skip.numel():
+            raise KernelError("gated_group_norm: the row is not a whole number of heads")
+        width = n // skip.numel()
+        x_ld = _row_slice(skip_x, "skip_x", torch.float32, T, n)
+    _work(_nbytes(y, out) + T * n * z.element_size() + (T * n * 4 if skip is not None else 0))
+    f = _fn("ssm", "llmie_gated_group_norm", [_c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_float, _c_void_p] +
+            [_c_int] * 4 + [_c_void_p, _c_int, _c_void_p, _c_int, _c_void_p])
+    _check(f(y.data_ptr(), z.data_ptr(), z_ld, _dt(z, "z"), weight.data_ptr(), float(eps), out.data_ptr(), _dt(out, "out"),
+             T, n, groups, _ptr(skip_x) if skip is not None else None, x_ld, _ptr(skip), width, _stream()),
+           "gated_group_norm")
     return out
 
 

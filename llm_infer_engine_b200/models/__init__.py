@@ -1,4 +1,4 @@
-from . import burinex, dofipel, ganupel, llama, zemivik  # noqa: F401  (register LlamaForCausalLM, Zemivik, Dofipel, Ganupel, Burinex)
+from . import burinex, dofipel, ganupel, llama, rogizen, zemivik  # noqa: F401  (register the architectures)
 from .decoder import DecoderModel
 
 __all__ = ["DecoderModel"]

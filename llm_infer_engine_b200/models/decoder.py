@@ -38,6 +38,7 @@ class DecoderModel:
         self.final_norm = build_part("norm", spec.final_norm, runtime)
         self.after_embedding = build_part("pointwise", spec.after_embedding, runtime) if spec.after_embedding else None
         self.after_head = build_part("pointwise", spec.after_head, runtime) if spec.after_head else None
+        self.stages = {name: build_part("stream", ps, runtime) for name, ps in spec.stages.items()}
         self.embedding: torch.Tensor = None
         self.head: Linear = None
 
@@ -63,6 +64,7 @@ class DecoderModel:
             out.append((self.spec.after_embedding_name, self.after_embedding))
         if self.after_head is not None:
             out.append((self.spec.after_head_name, self.after_head))
+        out.extend(self.stages.items())
         return out
 
     @staticmethod
@@ -98,6 +100,8 @@ class DecoderModel:
         total = self.head.nbytes() + self.final_norm.weight_bytes()
         for call in self.spec.schedule:
             total += sum(p.weight_bytes() for p in self.blocks[call.layer].parts().values())
+            if call.before is not None:
+                total += self.stages[call.before].weight_bytes()
         return total
 
     # ------------------------------------------------------------------ one step
@@ -107,6 +111,8 @@ class DecoderModel:
         ops.embedding(ctx.tokens, self.embedding, h)
         if self.after_embedding is not None:
             h = self.after_embedding.forward(h, ctx)
+        for stage in self.stages.values():
+            stage.begin(h, ctx)
         trace.pop()
         pending = None
         trace.push("Layers")
@@ -114,6 +120,8 @@ class DecoderModel:
             unit = cache.unit(self.unit_of_entry[pos])
             ctx.entry = pos
             block = self.blocks[call.layer]
+            if call.before is not None:
+                h, pending = self.stages[call.before].forward(h, pending, ctx)
             if isinstance(pending, DeferredBranchAdd) and not getattr(block, "accepts_deferred_branch_add", False):
                 h, pending = pending.apply(), None      # this block does not know deferred adds: done here
             h, pending = block.forward(h, pending, ctx, unit, call.cache_of is None)

@@ -1,6 +1,6 @@
 """Interfaces and registries of the parts a layer is put together from.
 
-Six kinds of part, each with a registry from a kind name to a class:
+Seven kinds of part, each with a registry from a kind name to a class:
 
     mixer              x[T, d] -> [T, d], mixes information between positions; may own cache
     feed_forward       x[T, d] -> [T, d], position-wise
@@ -10,6 +10,7 @@ Six kinds of part, each with a registry from a kind name to a class:
                        slots outside the layers (after the embedding, after the head)
     block              the arrangement of a layer's parts around the residual stream; it declares the
                        roles it has (`ROLES`) and the part group of each
+    stream             a stage between layers: it replaces the residual stream before a layer of the run order
 
 A part is constructed from `(params, runtime)`: `params` is the mapping of its `PartSpec`
 (every size and constant it needs; nothing is read from a model-wide config), `runtime` says
@@ -56,6 +57,7 @@ class AttentionOptions:
     knows it (the plain kernel first), so the call sites of the existing options do not change."""
     scale: float
     window: int = 0              # 0 = every earlier key; n = the last n keys, the token's own included
+    chunk: int = 0               # n > 0: only the keys of the token's own chunk of n positions, counted from position 0
     keep_first: int = 0          # with a window: the first n keys of the sequence stay visible behind it
     sink: bool = False           # one more term exp(0) in the softmax's denominator (a key of score 0, no value)
     sink_values: Optional[torch.Tensor] = None   # float32 [query heads]: the sink's score per head instead of 0
@@ -68,8 +70,14 @@ class AttentionOptions:
     sigmoid_bias: Optional[torch.Tensor] = None
 
     @property
+    def reach(self) -> int:
+        """How far back a token sees, in the form the attention kernels take: 0 = every earlier key, n > 0 = a window
+        of n keys, -n < 0 = its own chunk of n positions."""
+        return -self.chunk if self.chunk else self.window
+
+    @property
     def plain(self) -> bool:
-        """Only the options every attention kernel knows (scale, window)."""
+        """Only the options every attention kernel knows (scale, window, chunk)."""
         return self.keep_first == 0 and not self.sink and not self.scored and self.sigmoid_bias is None
 
     @property
@@ -123,17 +131,18 @@ class Norm(Part):
 
 
 class ScaledDelta:
-    """Branch output that is scaled on its way into the stream: vector (.) (c1 t1 + c2 t2), with `terms` a list of
-    one or two (tensor, constant) pairs and `vector` a float32 [d] scale per channel or None. A mixer made of two
+    """Branch output that is scaled on its way into the stream: vector (.) (c1 t1 + c2 t2) + bias, with `terms` a list of
+    one or two (tensor, constant) pairs, `vector` a float32 [d] scale per channel or None and `bias` a float32 [d] vector
+    (the bias of a branch's last product) or None. A mixer made of two
     mixers returns one without a vector; a block with a learned scale per channel puts its vector on whatever its
     branch returned. A norm whose kernel knows the form adds it while it reads the stream; `materialize()` gives the
     plain float32 tensor to everything else."""
 
-    def __init__(self, terms, vector: Optional[torch.Tensor] = None):
+    def __init__(self, terms, vector: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None):
         terms = [(t, float(c)) for t, c in terms]
         if not 1 <= len(terms) <= 2:
             raise ValueError("a ScaledDelta has one or two terms")
-        self.terms, self.vector = terms, vector
+        self.terms, self.vector, self.bias = terms, vector, bias
 
     @staticmethod
     def of(y, vector: Optional[torch.Tensor]) -> "ScaledDelta":
@@ -141,14 +150,21 @@ class ScaledDelta:
         if isinstance(y, ScaledDelta):
             if y.vector is not None:
                 raise ValueError("this branch output already carries a vector")
-            return ScaledDelta(y.terms, vector)
+            return ScaledDelta(y.terms, vector, None if y.bias is None else (y.bias * vector).contiguous())
         return ScaledDelta([(y, 1.0)], vector)
 
-    def materialize(self) -> torch.Tensor:
+    def add_into(self, h: torch.Tensor, out: Optional[torch.Tensor] = None, weight: Optional[torch.Tensor] = None,
+                 eps: float = 0.0, rows: Optional[torch.Tensor] = None) -> None:
+        """h (float32 [T, d]) += this, in place; `out`, if given, receives the new rows normed with `weight`, or as they
+        are without one. With `rows` only those rows are produced and h is untouched."""
         from ..kernels import ops
         (t1, c1), (t2, c2) = self.terms[0], (self.terms[1] if len(self.terms) > 1 else (None, 0.0))
-        out = torch.zeros(t1.shape, dtype=torch.float32, device=t1.device)
-        ops.scaled_add_rmsnorm(out, t1, c1, t2, c2, self.vector, None, 0.0, None)
+        ops.scaled_add_rmsnorm(h, t1, c1, t2, c2, self.vector, weight, eps, out, rows, bias=self.bias)
+
+    def materialize(self) -> torch.Tensor:
+        t = self.terms[0][0]
+        out = torch.zeros(t.shape, dtype=torch.float32, device=t.device)
+        self.add_into(out)
         return out
 
 
@@ -273,6 +289,19 @@ class Pointwise(Part):
         raise NotImplementedError
 
 
+class StreamStage(Part):
+    """A stage between layers, which the run order names before one of its entries (`LayerCall.before`): it replaces the
+    residual stream, for instance by a projection of it. `begin` is called once a step, right after the embedding and its
+    stage; what it wants to keep for the step goes into `ctx.carry`."""
+
+    def begin(self, h: torch.Tensor, ctx) -> None:
+        pass
+
+    def forward(self, h: torch.Tensor, pending, ctx):
+        """h float32 [T, d] and the branch output not yet added to it (see Block.forward) -> (new h, new pending)."""
+        raise NotImplementedError
+
+
 def call_branch(part, x, ctx, *cache_args, residual: Optional[torch.Tensor] = None):
     """Calls a mixer or feed-forward the way its class flags ask for: `residual` is passed only to a part
     that declared `adds_to_residual`, and a DeferredNorm is applied first unless the part accepts one."""
@@ -333,7 +362,7 @@ class Block:
 
 
 _REGISTRIES: Dict[str, Dict[str, type]] = {"mixer": {}, "feed_forward": {}, "norm": {}, "position_encoding": {},
-                                           "pointwise": {}, "block": {}}
+                                           "pointwise": {}, "block": {}, "stream": {}}
 
 
 def _register(group: str, kind: str, cls: type) -> None:
@@ -362,6 +391,10 @@ def register_pointwise(kind: str, cls: type) -> None:
 
 def register_block(kind: str, cls: type) -> None:
     _register("block", kind, cls)
+
+
+def register_stream(kind: str, cls: type) -> None:
+    _register("stream", kind, cls)
 
 
 def lookup(group: str, kind: str) -> type:

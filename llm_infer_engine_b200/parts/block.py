@@ -42,6 +42,22 @@ class PreNormBlock(Block):
 register_block("pre_norm", PreNormBlock)
 
 
+class PreNormMixerBlock(Block):
+    """The same arrangement for a layer without a feed-forward: h += mixer(norm(h))."""
+    ROLES = {"mixer": "mixer", "mixer_norm": "norm"}
+
+    def forward(self, h, pending, ctx, unit, owns_cache):
+        x = None
+        if pending is None and self.mixer.accepts_deferred_norm:
+            x = self.mixer_norm.defer(h)
+        if x is None:
+            x = self.mixer_norm.forward(h, pending)
+        return h, call_branch(self.mixer, x, ctx, unit, owns_cache, residual=h)
+
+
+register_block("pre_norm_mixer", PreNormMixerBlock)
+
+
 class BranchNormBlock(Block):
     """h += norm(mixer(h)); h += norm(feed_forward(h)): the branches read the residual stream itself and the norm
     sits on each branch's OUTPUT. The sum stays float32; a bfloat16 engine's products read the stream rounded to

@@ -17,6 +17,16 @@ import torch
 from ..kernels import ops
 
 
+ROW_TILE = 16      # rows of a weight that this library's products work on at a time
+
+
+def pad_rows(w: torch.Tensor) -> torch.Tensor:
+    """`w` [n, k] with rows of zeros up to a whole number of tiles: the products then take every n, and rows of the result
+    start on 16 bytes. The extra columns of the result are zeros."""
+    extra = -w.shape[0] % ROW_TILE
+    return w if not extra else torch.cat([w, torch.zeros((extra, w.shape[1]), dtype=w.dtype, device=w.device)])
+
+
 class Linear:
     def __init__(self, weight: torch.Tensor):
         if weight.dim() != 2:
@@ -48,15 +58,26 @@ class Linear:
                                    else ops.STREAM_STORE_BF16)
         return ops.library_mm(xb, w, out_dtype)
 
-    def add_into(self, x: torch.Tensor, h: torch.Tensor) -> bool:
-        """h (float32 [T, out]) += x W^T inside the product's kernel, when a kernel for this shape
+    def after_norm(self, x) -> Optional[torch.Tensor]:
+        """norm(h) W^T in float32 with the norm folded into the product's kernel, for a DeferredNorm `x` of one-token
+        steps; None when no kernel does that for this weight."""
+        if x.kind != "rmsnorm" or self.weight.dtype != torch.bfloat16 or self.out_features % ROW_TILE:
+            return None
+        out = torch.empty((x.shape[0], self.out_features), dtype=torch.float32, device=x.h.device)
+        return ops.norm_gemm_f32(x.h, x.weight, x.eps, self.weight, out)
+
+    def add_into(self, x: torch.Tensor, h: torch.Tensor, bias: Optional[torch.Tensor] = None) -> bool:
+        """h (float32 [T, out]) += x W^T (+ bias) inside the product's kernel, when a kernel for this shape
         exists. Returns False (and does nothing) otherwise."""
         if self.weight.dtype != torch.bfloat16 or x.dtype != torch.bfloat16:
             return False
         if not ops.gemm_skinny_add_wins(x.shape[0], self.out_features, self.in_features, x.device) \
                 or not ops.gemm_skinny_ok(x.shape[0], self.out_features, self.in_features):
             return False
-        ops.gemm_skinny(x, self.weight, h, ops.SKINNY_ADD_F32)
+        if bias is None:
+            ops.gemm_skinny(x, self.weight, h, ops.SKINNY_ADD_F32)
+        else:
+            ops.gemm_skinny_add_bias(x, self.weight, h, bias)
         return True
 
     def gated(self, x: torch.Tensor, act: int) -> Optional[torch.Tensor]:

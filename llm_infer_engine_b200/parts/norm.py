@@ -56,13 +56,16 @@ class RMSNorm(Norm):
         trace.push("RMSNorm")
         if isinstance(delta, ScaledDelta):
             # a scaled branch output (or two): the add, the scales and the norm are one kernel
-            (t1, c1), (t2, c2) = delta.terms[0], (delta.terms[1] if len(delta.terms) > 1 else (None, 0.0))
-            ops.scaled_add_rmsnorm(h, t1, c1, t2, c2, delta.vector, self.weight, self.eps, out, rows)
+            delta.add_into(h, out, self.weight, self.eps, rows)
             trace.pop()
             return out
         delta = single_delta(delta)
         if delta is not None and delta.dtype != out.dtype:
-            # the fused kernel adds a branch output of the activations' type; any other is added by a kernel of its own
+            # a branch output that is not of the activations' type: the kernel that takes either type
+            if self.size <= ops.SCALED_ADD_MAX_WIDTH:
+                ops.scaled_add_rmsnorm(h, delta, 1.0, None, 0.0, None, self.weight, self.eps, out, rows)
+                trace.pop()
+                return out
             if rows is not None:
                 h = h.clone()
             ops.residual_add(h, delta)

@@ -478,6 +478,25 @@ def burinex_config(width: int, heads: int, kv_heads: int, head_dim: int, ff: int
             "norm": {"eps": 1e-6}, "layers": layers}
 
 
+def rogizen_config(width: int, heads: int, kv_heads: int, head_dim: int, ff: int, vocab: int, n_layers: int,
+                   chunk: int) -> dict:
+    """A Rogizen configuration with a Llama shape's layer sizes. Layers cycle through four kinds: attention in chunks (4
+    taps, whole heads rotated with YaRN-scaled frequencies) + feed-forward, a state space layer (twice the width inside,
+    heads of 64 columns over 128 state rows, one group, 4 taps) + feed-forward, the same without a feed-forward, attention
+    + feed-forward. All layers form the loop, of one pass, so that as many layers run as in the other design."""
+    attn = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "conv": 4, "scale": head_dim ** -0.5,
+            "mask": {"size": chunk} if chunk else None,
+            "rot": {"base": 10000.0, "dims": head_dim,
+                    "scaling": {"factor": 8.0, "original": 2048, "fast": 16.0, "slow": 2.0}}}
+    ssm = {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": 1, "norm_groups": 1, "conv": 4}
+    dense = {"kind": "dense", "ff": ff}
+    kinds = [("attention", attn, dense), ("mamba2", ssm, dense), ("mamba2", ssm, None), ("attention", attn, dense)]
+    layers = [{"type": k, "mixer": json.loads(json.dumps(m)), "mlp": f} for k, m, f in (kinds[i % 4] for i in range(n_layers))]
+    return {"architecture": "Rogizen", "vocab": vocab, "width": width, "embedding": {"scale": width ** 0.5},
+            "logit_softcap": 30.0, "norm": {"eps": 1e-6}, "loop": {"start": 0, "stop": n_layers, "times": 1},
+            "layers": layers}
+
+
 def step_tables(engine, pk: dict, title: str, batch: int = 8) -> str:
     """Per-kernel tables (eager steps, CUDA events) of a decode step at `batch` sequences and of a 2,048-token
     prompt."""
@@ -517,7 +536,8 @@ def step_tables(engine, pk: dict, title: str, batch: int = 8) -> str:
 
 def run_designs(args, pk: dict, which: str = "Zemivik") -> str:
     """Zemivik (or, with which="Dofipel", Dofipel with a window of 1,024) beside Llama at equal layer sizes, or, with
-    which="Ganupel" or "Burinex", that design beside Dofipel (random weights, bfloat16): decode throughput at batch 1, 8 and 64
+    which="Ganupel" or "Burinex", that design beside Dofipel, or, with which="Rogizen", that design beside Ganupel
+    (random weights, bfloat16): decode throughput at batch 1, 8 and 64
     after 512-token prompts (captured steps, device time), prefill throughput of one 2,048-token prompt, and the
     per-kernel tables of both. Zemivik once without a mask (the attention work of Llama's) and once with a window
     of 1,024 tokens that keeps the first four. The shared vocabulary is kept small so that the layers, not the
@@ -529,7 +549,8 @@ def run_designs(args, pk: dict, which: str = "Zemivik") -> str:
     vocab = 32000
     shapes = [("1B layer sizes", CONFIG_1B), ("8B layer sizes", CONFIG_8B)]
     steps = min(args.steps, 64)
-    lines = [f"{which} beside {'Dofipel' if which in ('Ganupel', 'Burinex') else 'Llama'} at equal layer sizes, {n_layers} layers, vocabulary {vocab}, bfloat16, random weights "
+    beside = {"Ganupel": "Dofipel", "Burinex": "Dofipel", "Rogizen": "Ganupel"}.get(which, "Llama")
+    lines = [f"{which} beside {beside} at equal layer sizes, {n_layers} layers, vocabulary {vocab}, bfloat16, random weights "
              f"(peaks: {pk['hbm_gbs']:.0f} GB/s, {pk['bf16_tflops']:.0f} TFLOP/s, {pk['source']}).", "",
              "| layer sizes | design | decode b1 tok/s | ms/step | decode b8 tok/s | ms/step | decode b64 tok/s | ms/step | "
              f"prefill {PREFILL_TOKENS} tok/s | ms |", "|---|---|---|---|---|---|---|---|---|---|"]
@@ -551,6 +572,9 @@ def run_designs(args, pk: dict, which: str = "Zemivik") -> str:
         if which == "Burinex":
             designs = [("Dofipel, window 1024", dofipel_config(d, hq, hkv, hd, ff, vocab, n_layers, 1024)),
                        ("Burinex, window 1024", burinex_config(d, hq, hkv, hd, ff, vocab, n_layers, 1024))]
+        if which == "Rogizen":
+            designs = [("Ganupel, window 1024", ganupel_config(d, hq, hkv, hd, ff, vocab, n_layers, 1024)),
+                       ("Rogizen, chunks of 1024", rogizen_config(d, hq, hkv, hd, ff, vocab, n_layers, 1024))]
         for design, cfg in designs:
             folder = scratch_folder("llmie_bench_design_")
             write_random_model(cfg, folder, seed=3, std=0.02)
@@ -672,9 +696,9 @@ def run_ours(args):
             with open(args.per_kernel_out, "w", encoding="utf-8") as f:
                 f.write(text + "\n")
         return 0
-    if args.designs or args.dofipel or args.ganupel or args.burinex:
-        text = run_designs(args, pk, "Burinex" if args.burinex else "Ganupel" if args.ganupel else
-                           "Dofipel" if args.dofipel else "Zemivik")
+    if args.designs or args.dofipel or args.ganupel or args.burinex or args.rogizen:
+        text = run_designs(args, pk, "Rogizen" if args.rogizen else "Burinex" if args.burinex else "Ganupel" if args.ganupel
+                           else "Dofipel" if args.dofipel else "Zemivik")
         print(text)
         if args.per_kernel_out:
             with open(args.per_kernel_out, "w", encoding="utf-8") as f:
@@ -856,6 +880,9 @@ def main():
                     help="the same comparison for Burinex (post-norm layers; latent attention with a query latent, a "
                          "window and a learned sink; gated attention with a query temperature; linear attention with a "
                          "decay per head; routed experts weighted on their input) beside Dofipel, the closest design")
+    ap.add_argument("--rogizen", action="store_true",
+                    help="the same comparison for Rogizen (attention in chunks behind a short convolution, state space "
+                         "layers, the embedding mixed into the stream) beside Ganupel, the closest design")
     ap.add_argument("--heads", type=int, default=32, help="query heads of --attention-sweep")
     ap.add_argument("--kv-heads", type=int, default=8, help="KV heads of --attention-sweep")
     ap.add_argument("--head-dim", type=int, default=64, choices=[64, 128], help="head size of --attention-sweep")

@@ -101,8 +101,10 @@ class KernelPlan:
             if gate is not None:
                 ops.sigmoid_gate(out, gate)
             return True
-        # head sizes that none of the kernels above takes
-        return self._attention_by_rows(ctx, q, kv, out, n_q, n_kv, head_dim, options, gate)
+        if options.chunk:
+            # head sizes that none of the kernels above takes
+            return self._attention_by_rows(ctx, q, kv, out, n_q, n_kv, head_dim, options, gate)
+        return False
 
     def _sigmoid_attention(self, ctx, q, kv, out, n_q, n_kv, head_dim, options, gate) -> bool:
         """Attention without a softmax (weights sigmoid(score + a number per head), not normalised). Prompts of the

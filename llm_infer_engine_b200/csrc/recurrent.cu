@@ -312,10 +312,9 @@ __global__ void act_columns_kernel(const T* __restrict__ proj, int ld, int off0,
 // ------------------------------------------------------------------------------------------ vector state
 constexpr int kMaxTaps = 16;
 
-// A thread is V adjacent channels over a run of `tile` consecutive packed tokens. x = proj[:, x_off + c] + x_bias; inputs
-// before the step come from conv_state [slots, K-1, C] (the last K-1 inputs of the sequence so far, zeros at its start).
-// The thread keeps the last K inputs in registers: a token that follows its predecessor in the same sequence loads ONE new
-// input, the first token of a run or of a sequence's piece loads all K. Oldest input first: a fixed order of summation.
+// A thread is V adjacent channels over a run of consecutive packed tokens. x = proj[:, x_off + c] + x_bias; inputs before
+// the step come from conv_state [slots, K-1, C] (the last K-1 inputs of the sequence so far, zeros at its start). Oldest
+// input first: a fixed order of summation.
 // `act`: an activation of the result. `single`: every sequence of the step brings one token, so a channel's inputs are
 // this thread's alone and it also writes the new conv_state (in other steps conv_state_store does).
 template <typename TP, int V>
@@ -337,88 +336,108 @@ __device__ __forceinline__ void conv_input(const TP* p, const float (&xb)[V], fl
   for (int e = 0; e < V; ++e) x[e] += xb[e];
 }
 
-template <typename TP, typename TO, int KM, int V>
+template <typename TO, int V>
+__device__ __forceinline__ void conv_output(TO* dst, const float (&a)[V]) {
+  if (V == 4 && sizeof(TO) == 4) {
+    *reinterpret_cast<float4*>(dst) = make_float4(a[0], a[1 % V], a[2 % V], a[3 % V]);
+  } else if (V == 4) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(a[0], a[1 % V]), hi = __floats2bfloat162_rn(a[2 % V], a[3 % V]);
+    uint2 raw;
+    raw.x = *reinterpret_cast<const unsigned*>(&lo);
+    raw.y = *reinterpret_cast<const unsigned*>(&hi);
+    *reinterpret_cast<uint2*>(dst) = raw;
+  } else {
+    dst[0] = from_f32<TO>(a[0]);
+  }
+}
+
+// TILE: tokens a thread works on. A tile that lies within one sequence (nearly all do) asks for its TILE + K - 1 inputs at
+// once; one that crosses from a sequence into the next goes token by token, with all K inputs of each.
+template <typename TP, typename TO, int KM, int V, int TILE>
 __global__ void causal_conv_kernel(const TP* __restrict__ proj, int ld, int x_off, const float* __restrict__ x_bias,
                                    const float* __restrict__ taps, const float* __restrict__ conv_bias,
                                    float* conv_state, const int* __restrict__ cu_q,
                                    const int* __restrict__ tok_seq, const int* __restrict__ seq_slot,
-                                   TO* __restrict__ u, int C, int K, int n_tokens, int tile, int act, int single) {
+                                   TO* __restrict__ u, int C, int K, int n_tokens, int act, int single) {
   pdl_launch_dependents();
-  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
   if (c >= C) return;
-  float tp[KM][V], w[KM][V], xb[V], cb[V];
+  float tp[KM][V], xb[V], cb[V];                      // tp[i]: the taps of the inputs i tokens back
+  auto load_v = [&](const float* src, float (&v)[V]) {          // weights: no kernel writes them
+    if (V == 4) {
+      const float4 r = *reinterpret_cast<const float4*>(src + c);
+      v[0] = r.x; v[1 % V] = r.y; v[2 % V] = r.z; v[3 % V] = r.w;
+    } else {
+      v[0] = src[c];
+    }
+  };
 #pragma unroll
-  for (int e = 0; e < V; ++e) {
+  for (int e = 0; e < V; ++e) xb[e] = cb[e] = 0.f;
 #pragma unroll
-    for (int k = 0; k < KM; ++k) tp[k][e] = k < K ? taps[(size_t)(c + e) * K + k] : 0.f;   // weights: no kernel writes them
-    xb[e] = x_bias ? x_bias[c + e] : 0.f;
-    cb[e] = conv_bias ? conv_bias[c + e] : 0.f;
-  }
+  for (int i = 0; i < KM; ++i)
+    if (i < K) load_v(taps + (size_t)(K - 1 - i) * C, tp[i]);
+  if (x_bias) load_v(x_bias, xb);
+  if (conv_bias) load_v(conv_bias, cb);
   pdl_wait();
-  const int ta = blockIdx.y * tile, tb = min(ta + tile, n_tokens);
-  int prev_seq = -1;
-  for (int t = ta; t < tb; ++t) {
-    const int seq = tok_seq[t];
-    const int p = t - cu_q[seq];                      // place within this step's piece of the sequence
-    if (seq != prev_seq || p == 0) {
-      const float* old = conv_state + (size_t)seq_slot[seq] * (K - 1) * C + c;
+  const int ta = blockIdx.x * TILE, tb = min(ta + TILE, n_tokens);
+  constexpr int W = KM - 1;
+  float x[TILE + W][V];                               // x[W + j]: the input of token t0 + j
+  // the rows in front of the tile are asked for with the tile's own, before it is known whose they are
+  {
+    const TP* src = proj + (size_t)ta * ld + x_off + c;
 #pragma unroll
-      for (int k = 0; k < KM; ++k) {
-        if (k < K) {
-          const int m = p - (K - 1 - k);              // w[k] is the input K-1-k tokens back
-          if (m >= 0) {
-            conv_input<TP, V>(proj + (size_t)(t - (K - 1 - k)) * ld + x_off + c, xb, w[k]);
-          } else {
+    for (int j = 0; j < TILE; ++j)
+      if (ta + j < tb) conv_input<TP, V>(src + (size_t)j * ld, xb, x[W + j]);
 #pragma unroll
-            for (int e = 0; e < V; ++e) w[k][e] = old[(size_t)(K - 1 + m) * C + e];
-          }
+    for (int i = 1; i < KM; ++i)
+      if (i < K && ta - i >= 0) conv_input<TP, V>(src - (size_t)i * ld, xb, x[W - i]);
+  }
+  const bool whole = TILE == 1 || tok_seq[ta] == tok_seq[tb - 1];
+  for (int t0 = ta; t0 < tb; t0 += whole ? TILE : 1) {
+    const int seq = tok_seq[t0];
+    const int p = t0 - cu_q[seq];                     // place within this step's piece of the sequence
+    const int n = whole ? tb - t0 : 1;
+    const TP* src = proj + (size_t)t0 * ld + x_off + c;
+    if (!whole) conv_input<TP, V>(src, xb, x[W]);
+    float* cs = conv_state + (size_t)seq_slot[seq] * (K - 1) * C + c;
+#pragma unroll
+    for (int i = 1; i < KM; ++i) {
+      if (i < K) {
+        if (p - i >= 0) {
+          if (!whole) conv_input<TP, V>(src - (size_t)i * ld, xb, x[W - i]);
+        } else {
+#pragma unroll
+          for (int e = 0; e < V; ++e) x[W - i][e] = cs[(size_t)(K - 1 + p - i) * C + e];
         }
       }
-      prev_seq = seq;
-    } else {
+    }
 #pragma unroll
-      for (int k = 0; k + 1 < KM; ++k)
-        if (k + 1 < K) {
+    for (int j = 0; j < TILE; ++j) {
+      if (j < n) {
+        float acc[V];
 #pragma unroll
-          for (int e = 0; e < V; ++e) w[k][e] = w[k + 1][e];
+        for (int e = 0; e < V; ++e) {
+          acc[e] = cb[e];
+#pragma unroll
+          for (int i = KM - 1; i >= 0; --i)
+            if (i < K) acc[e] = fmaf(tp[i][e], x[W + j - i][e], acc[e]);
         }
-      float x[V];
-      conv_input<TP, V>(proj + (size_t)t * ld + x_off + c, xb, x);
+        if (sizeof(TO) == 2 && act == 4) {            // silu in front of a store that keeps 8 bits of it
 #pragma unroll
-      for (int k = 0; k < KM; ++k)
-        if (k == K - 1) {
+          for (int e = 0; e < V; ++e) acc[e] = acc[e] * __fdividef(1.f, 1.f + __expf(-acc[e]));
+        } else {
 #pragma unroll
-          for (int e = 0; e < V; ++e) w[k][e] = x[e];
+          for (int e = 0; e < V; ++e) acc[e] = apply_act(acc[e], act);
         }
+        conv_output<TO, V>(u + (size_t)(t0 + j) * C + c, acc);
+      }
     }
-    float acc[V];
+    if (single) {                                     // K - 1 inputs, the oldest first
 #pragma unroll
-    for (int e = 0; e < V; ++e) {
-      acc[e] = cb[e];
+      for (int i = 0; i + 1 < KM; ++i)
+        if (i + 1 < K) {
 #pragma unroll
-      for (int k = 0; k < KM; ++k)
-        if (k < K) acc[e] = fmaf(tp[k][e], w[k][e], acc[e]);
-      acc[e] = apply_act(acc[e], act);
-    }
-    TO* dst = u + (size_t)t * C + c;
-    if (V == 4 && sizeof(TO) == 4) {
-      *reinterpret_cast<float4*>(dst) = make_float4(acc[0], acc[1 % V], acc[2 % V], acc[3 % V]);
-    } else if (V == 4) {
-      const __nv_bfloat162 lo = __floats2bfloat162_rn(acc[0], acc[1 % V]), hi = __floats2bfloat162_rn(acc[2 % V], acc[3 % V]);
-      uint2 raw;
-      raw.x = *reinterpret_cast<const unsigned*>(&lo);
-      raw.y = *reinterpret_cast<const unsigned*>(&hi);
-      *reinterpret_cast<uint2*>(dst) = raw;
-    } else {
-      dst[0] = from_f32<TO>(acc[0]);
-    }
-    if (single) {
-      float* cs = conv_state + (size_t)seq_slot[seq] * (K - 1) * C + c;
-#pragma unroll
-      for (int k = 0; k + 1 < KM; ++k)
-        if (k + 1 < K) {
-#pragma unroll
-          for (int e = 0; e < V; ++e) cs[(size_t)k * C + e] = w[k + 1][e];
+          for (int e = 0; e < V; ++e) cs[(size_t)(K - 2 - i) * C + e] = x[W - i][e];
         }
     }
   }
@@ -829,21 +848,29 @@ static void causal_conv_launch(const TP* proj, int ld, int x_off, const float* x
                                const float* conv_bias, float* conv_state, const int* cu_q, const int* tok_seq,
                                const int* seq_slot, TO* u, int n_tokens, int C, int K, int act, int single,
                                cudaStream_t stream) {
-  const bool by4 = K <= 4 && C % 4 == 0 && ld % 4 == 0 && x_off % 4 == 0 && aligned16(proj) && aligned16(u);
-  const int tile = n_tokens >= 1024 ? 16 : (n_tokens >= 64 ? 4 : 1);
+  const bool by4 = K <= 4 && C % 4 == 0 && ld % 4 == 0 && x_off % 4 == 0 && aligned16(proj) && aligned16(u) && aligned16(taps) &&
+                   (!x_bias || aligned16(x_bias)) && (!conv_bias || aligned16(conv_bias));
   const int units = by4 ? C / 4 : C;
   const int threads = units >= 128 ? 128 : ((units + 31) / 32) * 32;
-  const dim3 grid((units + threads - 1) / threads, (n_tokens + tile - 1) / tile), block(threads);
-  if (by4)
-    launch_k(causal_conv_kernel<TP, TO, 4, 4>, grid, block, 0, stream, proj, ld, x_off, x_bias, taps, conv_bias, conv_state,
-             cu_q, tok_seq, seq_slot, u, C, K, n_tokens, tile, act, single);
-  else
-    launch_k(causal_conv_kernel<TP, TO, kMaxTaps, 1>, grid, block, 0, stream, proj, ld, x_off, x_bias, taps, conv_bias,
-             conv_state, cu_q, tok_seq, seq_slot, u, C, K, n_tokens, tile, act, single);
+#define LLMIE_CONV_LAUNCH(KM, V, TILE)                                                                                   \
+  launch_k(causal_conv_kernel<TP, TO, KM, V, TILE>, dim3((n_tokens + TILE - 1) / TILE, (units + threads - 1) / threads), \
+           dim3(threads), 0, stream, proj, ld, x_off, x_bias, taps, conv_bias, conv_state, cu_q, tok_seq, seq_slot, u, C, \
+           K, n_tokens, act, single)
+  if (!by4) {
+    if (n_tokens >= 64 && !single) LLMIE_CONV_LAUNCH(kMaxTaps, 1, 4);
+    else LLMIE_CONV_LAUNCH(kMaxTaps, 1, 1);
+  } else if (single || n_tokens < 64) {
+    LLMIE_CONV_LAUNCH(4, 4, 1);
+  } else if (n_tokens < 512) {
+    LLMIE_CONV_LAUNCH(4, 4, 4);
+  } else {
+    LLMIE_CONV_LAUNCH(4, 4, 8);
+  }
+#undef LLMIE_CONV_LAUNCH
 }
 
 // proj [T, ld] of `dtype` with the convolution's input at column x_off (C columns); x_bias, conv_bias float32 [C] or
-// null; taps float32 [C, K] (the last column multiplies the current token); conv_state float32 [slots, K-1, C];
+// null; taps float32 [K, C] (the last row multiplies the current token); conv_state float32 [slots, K-1, C];
 // u [T, C] of u_dtype = act(convolution), act a code of apply_act. single != 0: every sequence brings one token and the
 // new conv_state is written too.
 extern "C" int llmie_causal_conv_ex(const void* proj, int ld, int x_off, const float* x_bias, const float* taps,
@@ -851,7 +878,7 @@ extern "C" int llmie_causal_conv_ex(const void* proj, int ld, int x_off, const f
                                     const int* seq_slot, void* u, int u_dtype, int n_tokens, int C, int K, int act,
                                     int single, int dtype, cudaStream_t stream) {
   if (n_tokens < 0 || C <= 0 || K <= 0 || x_off < 0 || ld < x_off + C || act < 0 || act > 4) return LLMIE_ERR_BAD_ARG;
-  if (K > kMaxTaps || n_tokens > 65535 * 16) return LLMIE_ERR_UNSUPPORTED_SIZE;
+  if (K > kMaxTaps || C > 65535 * 32) return LLMIE_ERR_UNSUPPORTED_SIZE;
   if (n_tokens == 0) return LLMIE_OK;
 #define LLMIE_CONV(TP, TO)                                                                                              \
   causal_conv_launch<TP, TO>((const TP*)proj, ld, x_off, x_bias, taps, conv_bias, conv_state, cu_q, tok_seq, seq_slot,  \

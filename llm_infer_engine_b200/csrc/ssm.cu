@@ -12,7 +12,7 @@
 //   ssm_scan           prompts of the bfloat16 engine on the tensor cores, 64 tokens at a time (below)
 //   gated_group_norm   (y + D x) silu(z), then a root mean square over each of several equal runs of columns, weight
 //
-// ssm_scan. Within a chunk of Q = 64 tokens, with cum_i = sum_(k <= i) -A dt_k (float32, from the chunk's start):
+// ssm_scan. Within a chunk of Q = 64 tokens, with cum_i = sum_(k <= i) -A dt_k (float32, from the chunk's start; kept in base 2):
 //   y_i   = sum_(j <= i) (C_i . B_j) exp(cum_i - cum_j) dt_j x_j  +  exp(cum_i) C_i^T S_prev  +  D x_i
 //   S_new = exp(cum_last) S_prev + sum_j B_j (exp(cum_last - cum_j) dt_j x_j)^T
 // three matrix products and one more for the scores. A block walks over one sequence's chunks in order for one head and
@@ -165,6 +165,12 @@ __device__ __forceinline__ void ssm_ldm_t(unsigned (&r)[4], unsigned addr) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
 }
+// 2^x by the special-function unit (relative error about 2^-22)
+__device__ __forceinline__ float ssm_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 // two floats as (high, low) pairs of bfloat16: v = high + low up to 2^-17 of v
 __device__ __forceinline__ void ssm_split(float v0, float v1, unsigned& hi, unsigned& lo) {
   const __nv_bfloat162 h = __floats2bfloat162_rn(v0, v1);
@@ -198,7 +204,10 @@ ssm_scan_kernel(const SsmArgs p, const __nv_bfloat16* __restrict__ xbc, TO* __re
   constexpr int MT = (NT + 63) / 64;                        // 16-row tiles of the state a warp owns
   constexpr int PT = PS / 8;                                // 8-column tiles of the values
   extern __shared__ __align__(16) unsigned char ssm_smem[];
-  __shared__ float s_cum[kSsmQ], s_dt[kSsmQ], s_half;
+  // per token of a chunk, for this chunk and the next in turn: the sum of the decays' logarithms (base 2), the step, and
+  // the weight of the token's x in the state after the chunk
+  __shared__ __align__(16) float2 s_tok[2][kSsmQ];
+  __shared__ float s_xw[2][kSsmQ];
   __nv_bfloat16* stage0 = reinterpret_cast<__nv_bfloat16*>(ssm_smem);
   __nv_bfloat16* xw_hi = stage0 + 2 * Tile::kStage;         // [64][XP] exp(cum_last - cum_j) dt_j x_j
   __nv_bfloat16* xw_lo = xw_hi + Tile::kX;
@@ -242,7 +251,42 @@ ssm_scan_kernel(const SsmArgs p, const __nv_bfloat16* __restrict__ xbc, TO* __re
   };
   issue(0, 0);
 
-  // the state: warp w owns rows w * 16 + mt * 64 .. + 15
+  // Warp 0 works out the steps of a chunk, two tokens a lane, one chunk ahead; their raw values are asked for another
+  // chunk ahead of that. Tokens beyond the piece: dt = 0, no decay.
+  const float A2 = -A * 1.4426950408889634f;
+  float raw0 = 0.f, raw1 = 0.f;
+  auto fetch_raw = [&](int chunk) {
+    const int t = t_begin + chunk * kSsmQ + 2 * lane;
+    if (t < t_end) raw0 = to_f32(graw[(size_t)t * p.ld]);
+    if (t + 1 < t_end) raw1 = to_f32(graw[(size_t)(t + 1) * p.ld]);
+  };
+  auto make_steps = [&](int chunk) {
+    const int t = t_begin + chunk * kSsmQ + 2 * lane, buf = chunk & 1;
+    const float d0 = t < t_end ? ssm_softplus(raw0 + dt_bias) : 0.f;
+    const float d1 = t + 1 < t_end ? ssm_softplus(raw1 + dt_bias) : 0.f;
+    const float l0 = A2 * d0, l1 = A2 * d1;
+    float sum = l0 + l1;                              // of this lane's two, then up to and including them
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float up = __shfl_up_sync(0xffffffffu, sum, o);
+      if (lane >= o) sum += up;
+    }
+    float before = __shfl_up_sync(0xffffffffu, sum, 1);
+    if (lane == 0) before = 0.f;
+    const float c0 = before + l0, c1 = c0 + l1;
+    const float last = __shfl_sync(0xffffffffu, c1, 31);
+    s_tok[buf][2 * lane] = make_float2(c0, d0);
+    s_tok[buf][2 * lane + 1] = make_float2(c1, d1);
+    s_xw[buf][2 * lane] = exp2f(last - c0) * d0;
+    s_xw[buf][2 * lane + 1] = exp2f(last - c1) * d1;
+  };
+  if (warp == 0) {
+    fetch_raw(0);
+    make_steps(0);
+    fetch_raw(1);
+  }
+
+  // the state: warp w owns rows w * 16 + mt * 64 .. + 15; as a product's operand it lies in shared memory in two halves
   float* st = p.state + ((size_t)p.seq_slot[seq] * p.H + h) * N * P + p0;
   float S[MT][PT][4];
 #pragma unroll
@@ -257,30 +301,7 @@ ssm_scan_kernel(const SsmArgs p, const __nv_bfloat16* __restrict__ xbc, TO* __re
         S[mt][pt][2 * e] = v.x;
         S[mt][pt][2 * e + 1] = v.y;
       }
-
-  const int lm_row = lane & 15, lm_hi = (lane >> 4) * 8;                       // ldmatrix: A from row-major rows
-  const int lt_r = (lane & 7) + ((lane >> 4) & 1) * 8, lt_c = ((lane >> 3) & 1) * 8;   // A from its transpose
-  const int lb_r = (lane & 7) + ((lane >> 4) & 1) * 8, lb_c = ((lane >> 3) & 1) * 8;   // B, two 8-column tiles, k contiguous
-  const int lv_r = (lane & 7) + ((lane >> 3) & 1) * 8, lv_c = ((lane >> 4) & 1) * 8;   // B, two 8-column tiles, n contiguous
-  for (int chunk = 0; chunk < n_chunks; ++chunk) {
-    const int t0 = t_begin + chunk * kSsmQ;
-    const __nv_bfloat16* Bs = stage0 + (chunk & 1) * Tile::kStage;
-    const __nv_bfloat16* Cs = Bs + Tile::kB;
-    const __nv_bfloat16* Xs = Cs + Tile::kB;
-    if (chunk + 1 < n_chunks) issue(chunk + 1, (chunk + 1) & 1);
-    // ---- the chunk's steps and the sums of their logarithms (tokens beyond the piece: dt = 0, no decay)
-    float cum = 0.f, dt = 0.f;
-    if (tid < kSsmQ) {
-      if (t0 + tid < t_end) dt = ssm_softplus(to_f32(graw[(size_t)(t0 + tid) * p.ld]) + dt_bias);
-      cum = -A * dt;
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float up = __shfl_up_sync(0xffffffffu, cum, o);
-        if (lane >= o) cum += up;
-      }
-      if (tid == 31) s_half = cum;
-    }
-    // ---- the state before the chunk as a product's operand
+  auto publish_state = [&]() {
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt) {
       const int n = warp * 16 + mt * 64 + g;
@@ -297,19 +318,33 @@ ssm_scan_kernel(const SsmArgs p, const __nv_bfloat16* __restrict__ xbc, TO* __re
           }
       }
     }
-    if (chunk + 1 < n_chunks) asm volatile("cp.async.wait_group 1;" ::: "memory");
-    else asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();                                         // s_half; every thread's copies of this chunk
-    if (tid < kSsmQ) {
-      s_cum[tid] = warp == 0 ? cum : cum + s_half;
-      s_dt[tid] = dt;
+  };
+  publish_state();
+
+  const int lm_row = lane & 15, lm_hi = (lane >> 4) * 8;                       // ldmatrix: A from row-major rows
+  const int lt_r = (lane & 7) + ((lane >> 4) & 1) * 8, lt_c = ((lane >> 3) & 1) * 8;   // A from its transpose
+  const int lb_r = (lane & 7) + ((lane >> 4) & 1) * 8, lb_c = ((lane >> 3) & 1) * 8;   // B, two 8-column tiles, k contiguous
+  const int lv_r = (lane & 7) + ((lane >> 3) & 1) * 8, lv_c = ((lane >> 4) & 1) * 8;   // B, two 8-column tiles, n contiguous
+  for (int chunk = 0; chunk < n_chunks; ++chunk) {
+    const int t0 = t_begin + chunk * kSsmQ;
+    const __nv_bfloat16* Bs = stage0 + (chunk & 1) * Tile::kStage;
+    const __nv_bfloat16* Cs = Bs + Tile::kB;
+    const __nv_bfloat16* Xs = Cs + Tile::kB;
+    const float2* tok = s_tok[chunk & 1];
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                                         // this chunk is here; nobody works on the one before any more
+    if (chunk + 1 < n_chunks) {
+      issue(chunk + 1, (chunk + 1) & 1);
+      if (warp == 0) {
+        make_steps(chunk + 1);
+        fetch_raw(chunk + 2);
+      }
     }
-    __syncthreads();
-    const float cum_last = s_cum[kSsmQ - 1];
+    const float cum_last = tok[kSsmQ - 1].x;
     // ---- x weighted for the state's update
     for (int i = tid; i < kSsmQ * (PS / 2); i += kSsmThreads) {
       const int r = i / (PS / 2), c = (i % (PS / 2)) * 2;
-      const float w = expf(cum_last - s_cum[r]) * s_dt[r];
+      const float w = s_xw[chunk & 1][r];
       const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(Xs + r * XP + c));
       unsigned hi, lo;
       ssm_split(w * x.x, w * x.y, hi, lo);
@@ -349,9 +384,9 @@ ssm_scan_kernel(const SsmArgs p, const __nv_bfloat16* __restrict__ xbc, TO* __re
       }
     }
     const int i_lo = warp * 16 + g, i_hi = i_lo + 8;
-    const float cum_lo = s_cum[i_lo], cum_hi = s_cum[i_hi];
+    const float cum_lo = tok[i_lo].x, cum_hi = tok[i_hi].x;
     {
-      const float e_lo = expf(cum_lo), e_hi = expf(cum_hi);
+      const float e_lo = ssm_exp2(cum_lo), e_hi = ssm_exp2(cum_hi);
 #pragma unroll
       for (int pt = 0; pt < PT; ++pt) {
         yc[pt][0] *= e_lo;
@@ -369,12 +404,16 @@ ssm_scan_kernel(const SsmArgs p, const __nv_bfloat16* __restrict__ xbc, TO* __re
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
           const int j = kk * 16 + half * 8 + 2 * t4;
-          const float c0 = s_cum[j], c1 = s_cum[j + 1], d0 = s_dt[j], d1 = s_dt[j + 1];
+          const float4 cd = *reinterpret_cast<const float4*>(tok + j);     // (sum, step) of tokens j and j + 1
           const float* s = sc[2 * kk + half];
-          const float w0 = j <= i_lo ? s[0] * (expf(cum_lo - c0) * d0) : 0.f;
-          const float w1 = j + 1 <= i_lo ? s[1] * (expf(cum_lo - c1) * d1) : 0.f;
-          const float w2 = j <= i_hi ? s[2] * (expf(cum_hi - c0) * d0) : 0.f;
-          const float w3 = j + 1 <= i_hi ? s[3] * (expf(cum_hi - c1) * d1) : 0.f;
+          float w0 = s[0] * (ssm_exp2(cum_lo - cd.x) * cd.y), w1 = s[1] * (ssm_exp2(cum_lo - cd.z) * cd.w);
+          float w2 = s[2] * (ssm_exp2(cum_hi - cd.x) * cd.y), w3 = s[3] * (ssm_exp2(cum_hi - cd.z) * cd.w);
+          if (kk == warp) {                                  // the diagonal tile: later tokens are not seen
+            w0 = j <= i_lo ? w0 : 0.f;
+            w1 = j + 1 <= i_lo ? w1 : 0.f;
+            w2 = j <= i_hi ? w2 : 0.f;
+            w3 = j + 1 <= i_hi ? w3 : 0.f;
+          }
           ssm_split(w0, w1, ah[2 * half], al[2 * half]);
           ssm_split(w2, w3, ah[2 * half + 1], al[2 * half + 1]);
         }
@@ -409,7 +448,7 @@ ssm_scan_kernel(const SsmArgs p, const __nv_bfloat16* __restrict__ xbc, TO* __re
     }
     __syncthreads();                                         // the weighted x is complete
     // ---- the state after the chunk
-    const float e_last = expf(cum_last);
+    const float e_last = ssm_exp2(cum_last);
     const unsigned bt_addr = (unsigned)__cvta_generic_to_shared(Bs + lt_r * NP + lt_c + warp * 16);
     const unsigned xh_addr = (unsigned)__cvta_generic_to_shared(xw_hi + lv_r * XP + lv_c);
     const unsigned xl_addr = (unsigned)__cvta_generic_to_shared(xw_lo + lv_r * XP + lv_c);
@@ -439,7 +478,7 @@ ssm_scan_kernel(const SsmArgs p, const __nv_bfloat16* __restrict__ xbc, TO* __re
         }
       }
     }
-    __syncthreads();                                         // this stage, the operands and the sums may be written again
+    publish_state();                                         // every warp has read the state before the chunk
   }
   if (!p.write_state) return;
 #pragma unroll
@@ -466,8 +505,8 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ y, const TZ* _
   __shared__ float red[32];
   pdl_launch_dependents();
   pdl_wait();
-  const size_t t = blockIdx.y;
-  const int c0 = blockIdx.x * size;
+  const size_t t = blockIdx.x;
+  const int c0 = blockIdx.y * size;
   const float* yr = y + t * n + c0;
   const TZ* zr = z + t * z_ld + c0;
   float ss = 0.f;
@@ -530,7 +569,7 @@ static int gated_group_norm_launch(const float* y, const void* z, int z_ld, cons
                    (reinterpret_cast<uintptr_t>(z) & (4 * sizeof(TZ) - 1)) == 0;
   int threads = (((by4 ? size / 4 : size) + 31) / 32) * 32;
   threads = threads > 256 ? 256 : threads;
-  const dim3 grid(groups, n_tokens), block(threads);
+  const dim3 grid(n_tokens, groups), block(threads);
   auto kernel = by4 ? gated_group_norm_kernel<TZ, TO, 4> : gated_group_norm_kernel<TZ, TO, 1>;
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -651,9 +690,8 @@ extern "C" int llmie_gated_group_norm(const float* y, const void* z, int z_ld, i
   if (n_tokens < 0 || n <= 0 || groups <= 0 || n % groups || z_ld < n || !w || (!skip_x) != (!skip_d) ||
       (skip_d && (P <= 0 || n % P || x_ld < n)))
     return LLMIE_ERR_BAD_ARG;
-  if ((size_t)(n / groups) * sizeof(float) > 200 * 1024 || groups > 0x7fffffff) return LLMIE_ERR_UNSUPPORTED_SIZE;
+  if ((size_t)(n / groups) * sizeof(float) > 200 * 1024 || groups > 65535) return LLMIE_ERR_UNSUPPORTED_SIZE;
   if (n_tokens == 0) return LLMIE_OK;
-  if (n_tokens > 65535) return LLMIE_ERR_UNSUPPORTED_SIZE;
 #define LLMIE_GGN(TZ, TO) \
   gated_group_norm_launch<TZ, TO>(y, z, z_ld, w, eps, out, n_tokens, n, groups, skip_x, x_ld, skip_d, P, stream)
   if (z_dtype == LLMIE_F32 && out_dtype == LLMIE_F32) return LLMIE_GGN(float, float);

@@ -1780,15 +1780,16 @@ def act_columns(proj, runs, act: int):
 
 def causal_conv(proj, x_off: int, x_bias, taps, conv_bias, conv_state, cu_q, tok_seq, seq_slot, out, act: int = ACT_NONE,
                 single: bool = False):
-    """out[t, c] = act(conv_bias[c] + sum_j taps[c, K-1-j] x[t-j, c]) with x = proj[:, x_off + c] + x_bias[c]; inputs from
+    """out[t, c] = act(conv_bias[c] + sum_j taps[K-1-j, c] x[t-j, c]) with x = proj[:, x_off + c] + x_bias[c]; inputs from
     before the step are the slot's conv_state (its last K-1 inputs, zeros at a sequence's start).
-    taps float32 [C, K]; conv_state float32 [slots, K-1, C] (None with K = 1); out [T, C] float32 or bfloat16. `single`:
+    taps float32 [K, C] (the last row multiplies the current token); conv_state float32 [slots, K-1, C] (None with K = 1);
+    out [T, C] float32 or bfloat16. `single`:
     every sequence of the step brings one token, and the new conv_state is written too (`conv_state_store` does it for
     other steps)."""
     T, C = out.shape
-    K = taps.shape[1]
+    K = taps.shape[0]
     _need(proj, "proj", None, (T, None))
-    _need(taps, "taps", torch.float32, (C, K))
+    _need(taps, "taps", torch.float32, (K, C))
     if K > 1:
         _need(conv_state, "conv_state", torch.float32, (None, K - 1, C))
     _need(out, "out")
@@ -1828,16 +1829,16 @@ def conv_qk_store(proj, bias, taps, conv_state, q_w, k_w, eps: float, table, rot
     """What stands between the q and k projections of a layer with a short convolution and its attention: bias, a causal
     convolution per channel over time, RMS norm per head, rotation of the first rot_dim channels in pairs (2i, 2i + 1), and
     the cache write; the stored values are the keys as the convolution leaves them. proj [T, >= C] holds the q heads and
-    then the k heads (C = (n_q + n_kv) head_dim), float32 or bfloat16; bias float32 [C] or None; taps float32 [C, K];
+    then the k heads (C = (n_q + n_kv) head_dim), float32 or bfloat16; bias float32 [C] or None; taps float32 [K, C];
     conv_state float32 [slots, K-1, C] (None with K = 1); q_w, k_w float32 [head_dim]; table float32 [positions,
     rot_dim / 2, 2] of (cos, sin); q_out [T, n_q head_dim] and the caches of one dtype. `single`: every sequence brings one
     token, and the new conv_state is written too (`conv_state_store` does it for other steps)."""
     T, ld = proj.shape
-    C, K = (n_q + n_kv) * head_dim, taps.shape[1]
+    C, K = (n_q + n_kv) * head_dim, taps.shape[0]
     _need(proj, "proj")
     if ld < C:
         raise KernelError(f"conv_qk_store: rows of {ld} elements cannot hold q and k ({C})")
-    _need(taps, "taps", torch.float32, (C, K))
+    _need(taps, "taps", torch.float32, (K, C))
     if bias is not None:
         _need(bias, "bias", torch.float32, (C,))
     if K > 1:

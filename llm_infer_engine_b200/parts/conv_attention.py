@@ -89,7 +89,8 @@ class ConvAttention(Mixer):
         self.proj = Linear(pad_rows(torch.cat([w.to(dtype) for w in ws], dim=0)))          # [q | k], whole tiles of rows
         self.o = Linear(tensors[n["o"]])
         f32 = lambda *names: torch.cat([tensors[n[k]].to(torch.float32) for k in names]).contiguous()     # noqa: E731
-        self.conv_w, self.q_w, self.k_w = f32("q_conv", "k_conv"), f32("q_norm"), f32("k_norm")
+        self.conv_w = f32("q_conv", "k_conv").t().contiguous()                             # taps [K, C]
+        self.q_w, self.k_w = f32("q_norm"), f32("k_norm")
         if self.bias:
             self.qk_bias, self.o_bias = f32("q_bias", "k_bias"), f32("o_bias")
 

@@ -157,7 +157,7 @@ class GatedRecurrentUnit(Mixer):
         self.o = Linear(tensors[n["o"]])
         f32 = lambda t: t.to(torch.float32).contiguous()                        # noqa: E731
         self.y_bias, self.x_bias = f32(tensors[n["y_bias"]]), f32(tensors[n["x_bias"]])
-        self.conv_w, self.conv_bias = f32(tensors[n["conv"]]), f32(tensors[n["conv_bias"]])
+        self.conv_w, self.conv_bias = f32(tensors[n["conv"]].t()), f32(tensors[n["conv_bias"]])      # taps [K, C]
         # per group the rows of Ra and then of Ri: one batched product gives both gates' pre-activations
         self.gate_w = torch.cat([f32(tensors[n["ra"]]), f32(tensors[n["ri"]])], dim=1).contiguous()   # [B, 2 bw, bw]
         self.ra_bias, self.ri_bias = f32(tensors[n["ra_bias"]]).reshape(-1), f32(tensors[n["ri_bias"]]).reshape(-1)

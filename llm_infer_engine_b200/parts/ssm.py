@@ -78,7 +78,7 @@ class StateSpaceMixer(Mixer):
         self.proj = Linear(pad_rows(tensors[n["in"]]))          # [z | x | B | C | raw steps], whole tiles of rows
         self.o = Linear(tensors[n["o"]])
         f32 = lambda k: tensors[n[k]].to(torch.float32).contiguous()                        # noqa: E731
-        self.conv_w, self.conv_bias, self.dt_bias = f32("conv"), f32("conv_bias"), f32("dt_bias")
+        self.conv_w, self.conv_bias, self.dt_bias = f32("conv").t().contiguous(), f32("conv_bias"), f32("dt_bias")
         self.A, self.skip, self.norm_w = torch.exp(f32("A_log")).contiguous(), f32("D"), f32("norm")
 
     def weight_bytes(self) -> int:

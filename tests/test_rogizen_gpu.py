@@ -223,7 +223,7 @@ def test_convolution_in_pieces_carries_its_inputs(dtype, channels, taps):
         x = torch.cat([proj[i][held[i]:held[i] + pieces[i]] for i in live]).to(DEV)
         single = all(pieces[i] == 1 for i in live)
         out = torch.empty(cu[-1], channels, dtype=dt if sum(held) % 2 else torch.float32, device=DEV)
-        ops.causal_conv(x, 8, xb.to(DEV), w.to(DEV), cb.to(DEV), state, i32(cu), i32(tok_seq), slots[live].contiguous(), out,
+        ops.causal_conv(x, 8, xb.to(DEV), w.t().contiguous().to(DEV), cb.to(DEV), state, i32(cu), i32(tok_seq), slots[live].contiguous(), out,
                         act=ops.ACT_SILU, single=single)
         if taps > 1 and not single:
             ops.conv_state_store(x, 8, xb.to(DEV), state, i32(cu), slots[live].contiguous(), len(live))

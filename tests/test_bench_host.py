@@ -66,3 +66,15 @@ def test_shapes_of_the_benchmark_set():
     for cfg in (bench.CONFIG_1B, bench.CONFIG_3B, bench.CONFIG_8B):
         arch, typed = load_config(cfg)
         assert arch.name == "LlamaForCausalLM" and typed.vocab_size == 128256
+
+
+def test_rogizen_configuration_of_the_comparison():
+    """As many layer runs as layers, of the shape's sizes, and one pass of the loop around them."""
+    from llm_infer_engine_b200.config import load_config
+    cfg = bench.rogizen_config(2048, 32, 8, 64, 8192, 32000, 4, 1024)
+    arch, typed = load_config(cfg)
+    spec = arch.to_spec(typed)
+    assert arch.name == "Rogizen" and [c.layer for c in spec.schedule] == [0, 1, 2, 3]
+    assert spec.schedule[0].before == "loop" and not any(c.before for c in spec.schedule[1:])
+    assert typed.layers[1].mixer.heads * typed.layers[1].mixer.vdim == 2 * 2048 and typed.layers[2].ff is None
+    assert (typed.layers[0].mixer.chunk, typed.layers[0].ff) == (1024, 8192)

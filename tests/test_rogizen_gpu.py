@@ -633,6 +633,28 @@ def test_trace_run_program_and_other_sizes_at_once(tmp_path):
         compare(got, want, dtype, f"trace_run/{dtype}")
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_a_prompt_length_that_comes_again_is_replayed_right(dtype):
+    """Lone prompts of one length run eagerly, are captured, and are replayed, in other slots and at other start positions:
+    the convolution's inputs, the states, the loop's projection and the chunks inside the captured step."""
+    tag = "c"
+    engine = engine_for(tag, dtype, cuda_graph=True)
+    toks = [helpers.random_tokens(CFGS[tag]["vocab"], 90, seed=90 + i) for i in range(3)]
+    want = oracle(tag, {str(i): t for i, t in enumerate(toks)})
+    held = [engine.open() for _ in range(2)]                 # so that the slots differ from call to call
+    for i, t in enumerate(toks):
+        slot = engine.open()
+        for lo in (0, 30, 60):                               # three pieces of one length
+            got = engine.step([slot], [t[lo:lo + 30]], "last").float().cpu()[0]
+            ref = want[str(i)][lo + 29]
+            assert float((got - ref).abs().max()) <= bound(dtype, want[str(i)]), (i, lo)
+        if i == 0:
+            engine.close(held.pop())
+        engine.close(slot)
+    assert any(g for g in engine._prefill_graphs.values())
+    engine.close(held.pop())
+
+
 @pytest.mark.parametrize("dtype,gap", [("float32", 1e-4), ("bfloat16", 0.3)])
 @pytest.mark.parametrize("graph", [True, False])
 def test_greedy_generation_through_the_library(dtype, gap, graph):

@@ -1,8 +1,8 @@
 // What stands between the q and k projections of an attention layer with a short convolution and its scores, in one
 // kernel. For token t, head h of q or k and channel c (D channels a head), with u = the projection plus its bias:
 //
-//   y_t[c] = sum_j taps[c, j] u_(t - K + 1 + j)[c]         a causal convolution per channel over time, zeros before the
-//                                                          sequence; inputs from before the step come from the slot's state
+//   y_t[c] = sum_(i < K) f_i[c] u_(t - i)[c]               a causal convolution per channel over time; inputs from before the
+//                                                          step come from the slot's state (zeros in a new slot)
 //   values = y                                             key heads only: the values ARE the keys as they stand here
 //   n[c]   = y[c] / sqrt(mean_c(y^2) + eps) * w[c]         RMS norm per head, one weight [D] for all q heads, one for k
 //   rotation of the first `rot` channels in pairs (2i, 2i + 1) by the token's position, (cos, sin) from a table

@@ -2,7 +2,7 @@
 // and a state S [N, P] (float32, zero at a sequence's start, carried per slot), group g = h / (H / G):
 //
 //   dt_t = softplus(raw_t + dt_bias)          a_t = exp(-A dt_t),  A > 0 a number per head
-//   S_t  = a_t S_(t-1) + dt_t B_t x_t^T       y_t = S_t^T C_t + D x_t            B, C [N] shared by a group's heads
+//   S <- a_t S + B_t (dt_t x_t)^T              y_t = S^T C_t + D x_t              B, C [N] shared by a group's heads
 //
 // x, B and C are columns of one buffer xbc [T, H P + 2 G N] (what the convolution in front leaves), raw is a column of the
 // input projection, and so is z of the gated norm.

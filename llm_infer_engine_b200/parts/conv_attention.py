@@ -4,7 +4,8 @@ themselves.
 With h the layer's input [T, d], H query heads and G key heads of size D (query head i reads key head i // (H / G)), K taps:
 
     u = h W^T + b                            for q and for k: one product over row-concatenated weights
-    y_t = sum_j taps[:, j] u_(t - K + 1 + j)     per channel, zeros before the sequence's start (K = 1: a factor)
+    y_t = c_0 u_t + c_1 u_(t-1) + .. + c_(K-1) u_(t-K+1)     per channel; inputs from before the first token count as 0;
+                                             the checkpoint stores a channel's factors oldest first (K = 1: one factor)
     v = y                                    of the key heads: there is no value projection
     q, k <- y / sqrt(mean_head(y^2) + eps) * w   RMS norm per head, one weight [D] for all q heads and one for all k heads
     q, k <- rotated: entries (2i, 2i + 1) of the first `rot_dims` of a head by the position's angle (YaRN's frequencies and

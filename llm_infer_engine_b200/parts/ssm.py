@@ -3,10 +3,10 @@
 With h the layer's input [T, d], H heads of P value columns, a state of N rows, G groups of heads, K taps:
 
     z | x | B | C | raw = h W^T              widths H P, H P, G N, G N, H; one product
-    x | B | C <- silu(conv(x | B | C) + b)   causal, per channel, the last tap is the current token's; zeros before the start
+    x | B | C <- silu(conv(x | B | C) + b)   each channel's last K values, a token's own under the last of the stored taps
     dt = softplus(raw + dt_bias)             per token and head
-    S_t = exp(-exp(A_log) dt) S_(t-1) + dt B_t x_t^T         S [N, P] per head from zero; head i reads group i // (H / G)
-    y_t = S_t^T C_t + D x_t                  read from the NEW state
+    S   <- a S + B (dt x)^T,  a = exp(-A dt),  A = exp(A_log)    S [N, P] per head from zero; head i reads group i // (H / G)
+    y   = S^T C + D x                        read from the NEW state
     y   = norm(y silu(z)) * w                the gate comes first; the norm in `norm_groups` equal runs of columns
     out = y Wo^T
 

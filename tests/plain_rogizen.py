@@ -21,7 +21,8 @@ def silu(z):
 
 
 def short_conv(u, taps):
-    """y_t = sum_j taps[:, j] u_(t - K + 1 + j) per channel, u before the sequence = 0. u [T, C], taps [C, K]."""
+    """Per channel, token t gets the K inputs up to its own, each times its tap (taps [C, K], oldest first); what lies
+    before the first of u's [T, C] rows is 0."""
     T, K = u.shape[0], taps.shape[1]
     padded = torch.cat([torch.zeros(K - 1, u.shape[1], dtype=u.dtype), u])
     y = torch.zeros_like(u)
@@ -91,7 +92,7 @@ def attention(h, m, w, pre, eps):
 
 
 def state_space(xs, B, C, dt, A, D):
-    """S_t = exp(A dt_t) S_(t-1) + dt_t B_t x_t^T, y_t = S_t^T C_t + D x_t. xs [T, H, P], B and C [T, G, N] (head h reads
+    """S <- exp(A dt_t) S + B_t (dt_t x_t)^T from S = 0, then y_t = S^T C_t + D x_t. xs [T, H, P], B and C [T, G, N] (head h reads
     group h // (H / G)), dt [T, H], A and D [H]; returns y [T, H, P]."""
     T, H, P = xs.shape
     G, N = B.shape[1], B.shape[2]

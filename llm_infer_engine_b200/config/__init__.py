@@ -7,7 +7,9 @@ from .dofipel import DofipelConfig
 from .ganupel import GanupelConfig
 from .burinex import BurinexConfig
 from .rogizen import RogizenConfig
+from .selinex import SelinexConfig
 
 __all__ = ["Architecture", "ConfigError", "architecture_of", "known_architectures", "load_config",
            "read_config_json", "register_architecture", "LayerCall", "LayerSpec", "ModelSpec", "PartSpec",
-           "LlamaConfig", "RopeScaling", "ZemivikConfig", "DofipelConfig", "GanupelConfig", "BurinexConfig", "RogizenConfig"]
+           "LlamaConfig", "RopeScaling", "ZemivikConfig", "DofipelConfig", "GanupelConfig", "BurinexConfig", "RogizenConfig",
+           "SelinexConfig"]

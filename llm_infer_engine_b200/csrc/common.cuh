@@ -101,6 +101,20 @@ __device__ __forceinline__ float apply_act(float z, int act) {
   }
 }
 
+// What a gated feed-forward makes of a gate g and a linear part u: act(g) * u for the codes above, and with code 5 (only
+// here) both clamped and the linear part shifted: min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u, -limit, limit) + 1).
+struct GateForm {
+  int act;
+  float alpha, limit;
+};
+constexpr int kActClamped = 5;
+__device__ __forceinline__ float gated_pair(float g, float u, const GateForm& f) {
+  if (f.act != kActClamped) return apply_act(g, f.act) * u;
+  g = fminf(g, f.limit);
+  u = fminf(fmaxf(u, -f.limit), f.limit);
+  return g / (1.f + expf(-f.alpha * g)) * (u + 1.f);
+}
+
 // The first key a token at position `pos` may see, by the `window` argument of the attention kernels: 0 = every earlier
 // key; n > 0 = the last n keys, its own included; -n < 0 = the keys of its own chunk of n positions (chunks counted from
 // position 0 of the sequence).

@@ -50,7 +50,7 @@ __device__ __forceinline__ uint4 ldg16_stream(const void* p) {
 template <int NB, int EPI, int WARPS>
 __global__ void __launch_bounds__(WARPS * 32)
 skinny_gemm_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ W, void* __restrict__ out,
-                   int batch, int K, int ldo, int tile_stride, int hi_delta, const float* __restrict__ bias, int act) {
+                   int batch, int K, int ldo, int tile_stride, int hi_delta, const float* __restrict__ bias, GateForm act) {
   pdl_launch_dependents();
   __shared__ float red[WARPS][NB][16][8 + 1];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -179,7 +179,7 @@ skinny_gemm_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __r
         up += red[w][nb][j + 8][col];
       }
       // act 0: silu, the form this epilogue began with; any other activation code is applied to the gate instead
-      const float gated = (act ? apply_act(gate, act) : gate / (1.f + expf(-gate))) * up;
+      const float gated = act.act ? gated_pair(gate, up, act) : gate / (1.f + expf(-gate)) * up;
       reinterpret_cast<__nv_bfloat16*>(out)[(size_t)b * ldo + lo + j] = __float2bfloat16_rn(gated);
     }
   } else {
@@ -196,14 +196,14 @@ skinny_gemm_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __r
       if (EPI == kStoreF32) reinterpret_cast<float*>(out)[o] = v;
       if (EPI == kAddF32) reinterpret_cast<float*>(out)[o] += bias ? v + bias[n] : v;
       if (EPI == kBiasAct)
-        reinterpret_cast<__nv_bfloat16*>(out)[o] = __float2bfloat16_rn(apply_act(bias ? v + bias[n] : v, act));
+        reinterpret_cast<__nv_bfloat16*>(out)[o] = __float2bfloat16_rn(apply_act(bias ? v + bias[n] : v, act.act));
     }
   }
 }
 
 template <int NB, int WARPS>
 static int launch_epi(int epi, const void* x, const void* W, void* out, int batch, int K, int ldo, int tiles,
-                      int tile_stride, int hi_delta, const float* bias, int act, cudaStream_t stream) {
+                      int tile_stride, int hi_delta, const float* bias, GateForm act, cudaStream_t stream) {
   const __nv_bfloat16* xp = (const __nv_bfloat16*)x;
   const __nv_bfloat16* wp = (const __nv_bfloat16*)W;
   switch (epi) {
@@ -234,7 +234,7 @@ static int launch_epi(int epi, const void* x, const void* W, void* out, int batc
 // overlap with their neighbours' loads.
 template <int NB>
 static int launch_nb(int epi, const void* x, const void* W, void* out, int batch, int K, int ldo, int tiles,
-                     int tile_stride, int hi_delta, const float* bias, int act, cudaStream_t stream) {
+                     int tile_stride, int hi_delta, const float* bias, GateForm act, cudaStream_t stream) {
   const int chunks = K / 32;
   // An SM holds about 16 of these warps (registers). Doubling the warps of a block must leave every block
   // resident at once: 192 tiles of 16 warps would run as 148 blocks and then 44.
@@ -258,8 +258,8 @@ extern "C" int llmie_gemm_skinny_max_batch(void) { return 32; }
 //          4: out bfloat16 [batch, ldo] = act(y + bias), bias float32 [N] or null, act a code of apply_act
 // Needs K % 32 == 0, N % 16 == 0 (epilogue 3: ff % 8 == 0), 16-byte aligned x and W.
 static int gemm_skinny_entry(const void* x, const void* W, void* out, int batch, int N, int K, int ldo, int epilogue,
-                             const float* bias, int act, cudaStream_t stream) {
-  if (batch < 0 || N <= 0 || K <= 0 || act < 0 || act > 4) return LLMIE_ERR_BAD_ARG;
+                             const float* bias, GateForm act, cudaStream_t stream) {
+  if (batch < 0 || N <= 0 || K <= 0 || act.act < 0 || act.act > kActClamped) return LLMIE_ERR_BAD_ARG;
   if (batch > 32) return LLMIE_ERR_UNSUPPORTED_SIZE;
   if (K % 32) return LLMIE_ERR_UNSUPPORTED_SIZE;
   if (!aligned16(x) || !aligned16(W)) return LLMIE_ERR_ALIGNMENT;
@@ -280,25 +280,26 @@ static int gemm_skinny_entry(const void* x, const void* W, void* out, int batch,
 extern "C" int llmie_gemm_skinny(const void* x, const void* W, void* out, int batch, int N, int K, int ldo,
                                  int epilogue, cudaStream_t stream) {
   if (epilogue == kBiasAct) return LLMIE_ERR_BAD_ARG;
-  return gemm_skinny_entry(x, W, out, batch, N, K, ldo, epilogue, nullptr, 0, stream);
+  return gemm_skinny_entry(x, W, out, batch, N, K, ldo, epilogue, nullptr, GateForm{0, 0.f, 0.f}, stream);
 }
 
 // out bfloat16 [batch, N / 2] = act(x Wg^T) * (x Wu^T) for W = [gate rows; up rows]: epilogue 3 with an activation of
-// the caller's choice (a code of common.cuh's apply_act; 0 = silu).
+// the caller's choice (a code of common.cuh's apply_act; 0 = silu; 5 with alpha and limit: common.cuh's gated_pair).
 extern "C" int llmie_gemm_skinny_gated(const void* x, const void* W, void* out, int batch, int N, int K, int ldo, int act,
-                                       cudaStream_t stream) {
-  if (act < 0 || act > 4) return LLMIE_ERR_BAD_ARG;
-  return gemm_skinny_entry(x, W, out, batch, N, K, ldo, kSwiGLU, nullptr, act == 4 ? 0 : act, stream);
+                                       float alpha, float limit, cudaStream_t stream) {
+  return gemm_skinny_entry(x, W, out, batch, N, K, ldo, kSwiGLU, nullptr, GateForm{act == 4 ? 0 : act, alpha, limit},
+                           stream);
 }
 
 // out float32 [batch, ldo] += x W^T + bias (bias float32 [N] or null).
 extern "C" int llmie_gemm_skinny_add_bias(const void* x, const void* W, void* out, int batch, int N, int K, int ldo,
                                           const float* bias, cudaStream_t stream) {
-  return gemm_skinny_entry(x, W, out, batch, N, K, ldo, kAddF32, bias, 0, stream);
+  return gemm_skinny_entry(x, W, out, batch, N, K, ldo, kAddF32, bias, GateForm{0, 0.f, 0.f}, stream);
 }
 
 // out bfloat16 [batch, ldo] = act(x W^T + bias) in one kernel.
 extern "C" int llmie_gemm_skinny_bias_act(const void* x, const void* W, void* out, int batch, int N, int K, int ldo,
                                           const float* bias, int act, cudaStream_t stream) {
-  return gemm_skinny_entry(x, W, out, batch, N, K, ldo, kBiasAct, bias, act, stream);
+  if (act < 0 || act > 4) return LLMIE_ERR_BAD_ARG;
+  return gemm_skinny_entry(x, W, out, batch, N, K, ldo, kBiasAct, bias, GateForm{act, 0.f, 0.f}, stream);
 }

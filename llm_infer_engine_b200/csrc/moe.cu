@@ -8,6 +8,9 @@
 //             (the correction steers the choice only); weights = the chosen scores / (their sum + 1e-20) * a constant
 //             third rule (`mode` 2): scores = sigmoid(z) one by one; the `top` largest are chosen and the weights are the
 //             chosen scores themselves (times a constant), not normalised
+//             fourth rule (`mode` 3): scores = sigmoid(z) one by one; choice scores = score + correction; experts form
+//             equal groups of neighbours, a group's score is the sum of its two largest choice scores, and only experts
+//             of the `keep` best groups can be chosen (ties: the lower index); weights as in the third rule
 //   gather    out[p] = weights[pair at p] * x[token at p] for the sorted positions p: for designs whose weight
 //             multiplies what the expert READS (the combine then adds the experts' outputs with weight one)
 //   sort      the (token, choice) pairs grouped by expert into tiles of `tile` positions, padded per expert; one block,
@@ -25,13 +28,13 @@ template <typename T>
 __global__ void __launch_bounds__(kRouteWarps * 32)
 moe_route_kernel(const T* __restrict__ x, const float* __restrict__ w, const float* __restrict__ bias,
                  int* __restrict__ ids, float* __restrict__ weights, int n_tokens, int d, int n_experts, int top,
-                 int mode, const float* __restrict__ correction, float out_scale) {
+                 int mode, const float* __restrict__ correction, float out_scale, int n_groups, int keep) {
   // A block per token: the token's row is staged once as float32, its warps share out the experts, and a warp's lanes
   // take fixed columns of a dot product (four running sums each, added in a fixed order).
   extern __shared__ __align__(16) float route_smem[];            // [d] the row | [n_experts] the logits | scores
   float* xs = route_smem;
   float* z = route_smem + d;
-  float* sc = z + n_experts;                                     // mode 1: the scores the weights are made of
+  float* sc = z + n_experts;                                     // modes 1, 3: the scores the weights are made of
   pdl_launch_dependents();
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -88,6 +91,33 @@ moe_route_kernel(const T* __restrict__ x, const float* __restrict__ w, const flo
     }
     __syncwarp();
   }
+  if (mode == 3) {
+    // scores and choice scores; then the groups' scores, and the experts of all but the best groups out of the choice
+    float* gs = sc + n_experts;
+    const int size = n_experts / n_groups;
+    for (int e = lane; e < n_experts; e += 32) {
+      const float p = 1.f / (1.f + expf(-z[e]));
+      sc[e] = p;
+      z[e] = p + (correction ? correction[e] : 0.f);
+    }
+    __syncwarp();
+    for (int gi = lane; gi < n_groups; gi += 32) {
+      float hi = -INFINITY, lo = -INFINITY;
+      for (int i = 0; i < size; ++i) {
+        const float v = z[gi * size + i];
+        if (v > hi) { lo = hi; hi = v; } else if (v > lo) { lo = v; }
+      }
+      gs[gi] = size > 1 ? hi + lo : hi;
+    }
+    __syncwarp();
+    for (int gi = lane; gi < n_groups; gi += 32) {
+      int better = 0;
+      for (int i = 0; i < n_groups; ++i) better += gs[i] > gs[gi] || (gs[i] == gs[gi] && i < gi);
+      if (better >= keep)
+        for (int i = 0; i < size; ++i) z[gi * size + i] = -INFINITY;
+    }
+    __syncwarp();
+  }
   float first = 0.f, denom = 0.f, mine = 0.f;      // lane k keeps the k-th chosen logit
   int mine_id = 0;
   for (int k = 0; k < top; ++k) {
@@ -104,7 +134,7 @@ moe_route_kernel(const T* __restrict__ x, const float* __restrict__ w, const flo
       if (ov > best || (ov == best && oe < best_e)) { best = ov; best_e = oe; }
     }
     if (k == 0) first = best;
-    const float p = mode == 1 ? (best_e < n_experts ? sc[best_e] : 0.f)
+    const float p = (mode & 1) ? (best_e < n_experts ? sc[best_e] : 0.f)
                     : mode == 2 ? 1.f / (1.f + expf(-best)) : expf(best - first);
     denom += p;
     if ((k & 31) == lane) { mine = p; mine_id = best_e; }
@@ -120,7 +150,7 @@ moe_route_kernel(const T* __restrict__ x, const float* __restrict__ w, const flo
     }
   }
   __syncwarp();
-  const float inv = mode == 1 ? out_scale / (denom + 1e-20f) : mode == 2 ? out_scale : 1.f / denom;
+  const float inv = mode == 1 ? out_scale / (denom + 1e-20f) : mode >= 2 ? out_scale : 1.f / denom;
   for (int k = lane; k < top; k += 32) weights[(size_t)t * top + k] *= inv;
 }
 
@@ -288,23 +318,38 @@ using namespace llmie;
 // x [T, d] of x_dtype; w float32 [E, d]; bias float32 [E] or null; ids int32 [T, top]; weights float32 [T, top].
 // mode 0: the rule above (bias added to the logits, softmax over the chosen logits). mode 1: softmax over all logits,
 // choice by score + correction (float32 [E] or null), weights = chosen scores / (their sum + 1e-20) * out_scale.
-// mode 2: weights = sigmoid of the chosen logits * out_scale, not normalised.
+// mode 2: weights = sigmoid of the chosen logits * out_scale, not normalised. mode 3: the same weights, the choice by
+// score + correction among the experts of the `keep` best of n_groups groups.
+extern "C" int llmie_moe_route_groups(const void* x, int x_dtype, const float* w, const float* bias, int* ids,
+                                      float* weights, int n_tokens, int d, int n_experts, int top, int mode,
+                                      const float* correction, float out_scale, int n_groups, int keep,
+                                      cudaStream_t stream) {
+  if (n_tokens < 0 || d <= 0 || n_experts <= 0 || top <= 0 || top > n_experts) return LLMIE_ERR_BAD_ARG;
+  if (mode < 0 || mode > 3) return LLMIE_ERR_BAD_ARG;
+  if (mode == 3 && (n_groups <= 0 || n_experts % n_groups || keep <= 0 || keep > n_groups ||
+                    top > n_experts / n_groups * keep))
+    return LLMIE_ERR_BAD_ARG;
+  if (x_dtype != LLMIE_F32 && x_dtype != LLMIE_BF16) return LLMIE_ERR_DTYPE;
+  const size_t smem = ((size_t)d + 2 * (size_t)n_experts + (mode == 3 ? (size_t)n_groups : 0)) * sizeof(float);
+  if (smem > 48 * 1024) return LLMIE_ERR_UNSUPPORTED_SIZE;
+  if (n_tokens == 0) return LLMIE_OK;
+  const dim3 grid(n_tokens), block(kRouteWarps * 32);
+  if (x_dtype == LLMIE_F32)
+    launch_k(moe_route_kernel<float>, grid, block, smem, stream, (const float*)x, w, bias, ids, weights, n_tokens, d,
+             n_experts, top, mode, correction, out_scale, n_groups, keep);
+  else
+    launch_k(moe_route_kernel<__nv_bfloat16>, grid, block, smem, stream, (const __nv_bfloat16*)x, w, bias, ids, weights,
+             n_tokens, d, n_experts, top, mode, correction, out_scale, n_groups, keep);
+  LLMIE_LAUNCH_CHECK();
+  return LLMIE_OK;
+}
+
 extern "C" int llmie_moe_route_ex(const void* x, int x_dtype, const float* w, const float* bias, int* ids,
                                   float* weights, int n_tokens, int d, int n_experts, int top, int mode,
                                   const float* correction, float out_scale, cudaStream_t stream) {
-  if (n_tokens < 0 || d <= 0 || n_experts <= 0 || top <= 0 || top > n_experts) return LLMIE_ERR_BAD_ARG;
-  if (mode < 0 || mode > 2) return LLMIE_ERR_BAD_ARG;
-  if (x_dtype != LLMIE_F32 && x_dtype != LLMIE_BF16) return LLMIE_ERR_DTYPE;
-  const size_t smem = ((size_t)d + 2 * (size_t)n_experts) * sizeof(float);
-  if (smem > 48 * 1024) return LLMIE_ERR_UNSUPPORTED_SIZE;
-  if (n_tokens == 0) return LLMIE_OK;
-  const int blocks = n_tokens;
-  if (x_dtype == LLMIE_F32)
-    launch_k(moe_route_kernel<float>, dim3(blocks), dim3(kRouteWarps * 32), smem, stream, (const float*)x, w, bias, ids, weights, n_tokens, d, n_experts, top, mode, correction, out_scale);
-  else
-    launch_k(moe_route_kernel<__nv_bfloat16>, dim3(blocks), dim3(kRouteWarps * 32), smem, stream, (const __nv_bfloat16*)x, w, bias, ids, weights, n_tokens, d, n_experts, top, mode, correction, out_scale);
-  LLMIE_LAUNCH_CHECK();
-  return LLMIE_OK;
+  if (mode == 3) return LLMIE_ERR_BAD_ARG;
+  return llmie_moe_route_groups(x, x_dtype, w, bias, ids, weights, n_tokens, d, n_experts, top, mode, correction, out_scale,
+                                1, 1, stream);
 }
 
 extern "C" int llmie_moe_route(const void* x, int x_dtype, const float* w, const float* bias, int* ids, float* weights,

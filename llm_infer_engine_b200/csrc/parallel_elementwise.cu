@@ -80,7 +80,7 @@ __global__ void add_dyt_vec_kernel(float* __restrict__ h, const TD* __restrict__
 }
 
 template <typename T>
-__global__ void gated_act_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int ff, int act, size_t total) {
+__global__ void gated_act_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int ff, GateForm form, size_t total) {
   pdl_launch_dependents();
   pdl_wait();
   size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -90,13 +90,13 @@ __global__ void gated_act_kernel(const T* __restrict__ gate_up, T* __restrict__ 
     const int j = (int)(i - t * ff);
     const float g = to_f32(gate_up[t * 2 * ff + j]);
     const float u = to_f32(gate_up[t * 2 * ff + ff + j]);
-    out[i] = from_f32<T>(apply_act(g, act) * u);
+    out[i] = from_f32<T>(gated_pair(g, u, form));
   }
 }
 
 // ff % 8 == 0, 16-byte aligned: eight outputs a thread, a row of blocks per token (no index is divided)
 template <typename T>
-__global__ void gated_act_vec_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int ff, int act) {
+__global__ void gated_act_vec_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int ff, GateForm form) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t t = blockIdx.y;
@@ -106,7 +106,7 @@ __global__ void gated_act_vec_kernel(const T* __restrict__ gate_up, T* __restric
     load8(row + j, g);
     load8(row + ff + j, u);
 #pragma unroll
-    for (int e = 0; e < 8; ++e) o[e] = apply_act(g[e], act) * u[e];
+    for (int e = 0; e < 8; ++e) o[e] = gated_pair(g[e], u[e], form);
     store8(out + t * ff + j, o);
   }
 }
@@ -174,23 +174,25 @@ extern "C" int llmie_add_dyt(float* h, const void* d1, int d1_dtype, const void*
   return LLMIE_OK;
 }
 
-// gate_up [T, 2 ff] = [gate | up] per row; out [T, ff]; both of `dtype`; act one of the activation codes.
-extern "C" int llmie_gated_act(const void* gate_up, void* out, int n_tokens, int ff, int act, int dtype,
-                               cudaStream_t stream) {
-  if (n_tokens < 0 || ff <= 0 || act < 0 || act > 4) return LLMIE_ERR_BAD_ARG;
+// gate_up [T, 2 ff] = [gate | up] per row; out [T, ff]; both of `dtype`; act one of the activation codes, or 5 with
+// alpha and limit (common.cuh: gated_pair).
+extern "C" int llmie_gated_act(const void* gate_up, void* out, int n_tokens, int ff, int act, float alpha, float limit,
+                               int dtype, cudaStream_t stream) {
+  if (n_tokens < 0 || ff <= 0 || act < 0 || act > kActClamped) return LLMIE_ERR_BAD_ARG;
   if (dtype != LLMIE_F32 && dtype != LLMIE_BF16) return LLMIE_ERR_DTYPE;
   if (n_tokens == 0) return LLMIE_OK;
+  const GateForm form{act, alpha, limit};
   const size_t total = (size_t)n_tokens * ff;
   const bool vec = ff % 8 == 0 && aligned16(gate_up) && aligned16(out) && n_tokens <= 65535;
   if (vec) {
     const int bx = (ff / 8 + 127) / 128;
     dim3 grid(bx, n_tokens);
-    if (dtype == LLMIE_F32) launch_k(gated_act_vec_kernel<float>, grid, dim3(128), 0, stream, (const float*)gate_up, (float*)out, ff, act);
-    else launch_k(gated_act_vec_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, ff, act);
+    if (dtype == LLMIE_F32) launch_k(gated_act_vec_kernel<float>, grid, dim3(128), 0, stream, (const float*)gate_up, (float*)out, ff, form);
+    else launch_k(gated_act_vec_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, ff, form);
   } else {
     const int blocks = sweep_blocks(total, 256);
-    if (dtype == LLMIE_F32) launch_k(gated_act_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)gate_up, (float*)out, ff, act, total);
-    else launch_k(gated_act_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, ff, act, total);
+    if (dtype == LLMIE_F32) launch_k(gated_act_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)gate_up, (float*)out, ff, form, total);
+    else launch_k(gated_act_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, ff, form, total);
   }
   LLMIE_LAUNCH_CHECK();
   return LLMIE_OK;

@@ -14,8 +14,8 @@
 //                      queries shared by groups of heads (a state space model)
 //   act_columns        float32 copies of up to three runs of columns of the projections, through an activation
 //   matrix_scan_chunked  the same for long pieces, cut into chunks that run side by side (below)
-//   head_rmsnorm       o / sqrt(mean(o^2) + eps) * w over each head's vdim (or over the whole row, with a weight per
-//                      column), optionally times sigmoid(gate)
+//   head_rmsnorm       o / sqrt(mean(o^2) + eps) * w over each head's vdim (or over the whole row), w shared by the heads
+//                      or with a weight per column, optionally times sigmoid(gate) or silu(gate)
 //   causal_conv        u_t = act(b + sum_j taps[:, K-1-j] x_(t-j)), x before the step from the state's last K-1 inputs
 //   conv_state_store   the last K-1 inputs after the step (a one-token step's causal_conv writes them itself)
 //   unit_gate_values   a = exp(-c r softplus(lam)), drive = sqrt(1 - a^2) i u, r and i sigmoids of given pre-activations
@@ -225,17 +225,22 @@ __global__ void matrix_scan_chain_kernel(const float* __restrict__ state, const 
   }
 }
 
+// sigmoid(z), or silu(z) = z sigmoid(z)
+__device__ __forceinline__ float gate_factor(float z, int silu) { return (silu ? z : 1.f) / (1.f + expf(-z)); }
+
 // a warp per (token, head): o float32 [T, H * Dv] -> y of the activation type. `gate` (rows gate_ld apart, null = none):
-// the result is multiplied by sigmoid(gate) of the same place. An item may also be a token's whole row (Dv = the row).
+// the result is multiplied by sigmoid(gate) (or silu) of the same place. An item may also be a token's whole row (Dv = the
+// row). The weights repeat every w_items items (1: all heads share them).
 template <typename T>
 __global__ void head_rmsnorm_kernel(const float* __restrict__ o, const float* __restrict__ w, float eps,
                                     T* __restrict__ y, int Dv, size_t n_items, const T* __restrict__ gate, int gate_ld,
-                                    int items_per_row) {
+                                    int items_per_row, int silu, int w_items) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t item = (size_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
   if (item >= n_items) return;
+  if (w_items > 1) w += (item % w_items) * Dv;
   const float* row = o + item * Dv;
   float ss = 0.f;
   for (int i = lane; i < Dv; i += 32) { const float x = row[i]; ss = fmaf(x, x, ss); }
@@ -248,7 +253,7 @@ __global__ void head_rmsnorm_kernel(const float* __restrict__ o, const float* __
   const size_t t = item / items_per_row;
   const T* gr = gate + t * gate_ld + (item - t * items_per_row) * Dv;
   for (int i = lane; i < Dv; i += 32)
-    y[item * Dv + i] = from_f32<T>(row[i] * r * w[i] / (1.f + expf(-to_f32(gr[i]))));
+    y[item * Dv + i] = from_f32<T>(row[i] * r * w[i] * gate_factor(to_f32(gr[i]), silu));
 }
 
 // The same for wide items (a token's whole row of concatenated heads): a block per item, so that a one-token step's few
@@ -256,11 +261,12 @@ __global__ void head_rmsnorm_kernel(const float* __restrict__ o, const float* __
 template <typename T>
 __global__ void __launch_bounds__(256)
 row_rmsnorm_kernel(const float* __restrict__ o, const float* __restrict__ w, float eps, T* __restrict__ y, int Dv,
-                   const T* __restrict__ gate, int gate_ld, int items_per_row) {
+                   const T* __restrict__ gate, int gate_ld, int items_per_row, int silu, int w_items) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float red[32];
   const size_t item = blockIdx.x;
+  if (w_items > 1) w += (item % w_items) * Dv;
   const float4* row = reinterpret_cast<const float4*>(o + item * Dv);
   const int n4 = Dv >> 2;
   float ss = 0.f;
@@ -279,7 +285,7 @@ row_rmsnorm_kernel(const float* __restrict__ o, const float* __restrict__ w, flo
     float v[4] = {x.x * r * wv.x, x.y * r * wv.y, x.z * r * wv.z, x.w * r * wv.w};
     if (gr) {
 #pragma unroll
-      for (int e = 0; e < 4; ++e) v[e] = v[e] / (1.f + expf(-to_f32(gr[4 * i + e])));
+      for (int e = 0; e < 4; ++e) v[e] = v[e] * gate_factor(to_f32(gr[4 * i + e]), silu);
     }
 #pragma unroll
     for (int e = 0; e < 4; ++e) yr[4 * i + e] = from_f32<T>(v[e]);
@@ -802,21 +808,22 @@ extern "C" int llmie_act_columns(const void* proj, int ld, int off0, int n0, flo
 }
 
 // o float32 [n_items, Dv] (an item = a token's head); w float32 [Dv]; y [n_items, Dv] of `dtype`.
-// gate (of `dtype`, rows gate_ld apart, items_per_row items a row) or null: y is also multiplied by sigmoid(gate).
-extern "C" int llmie_head_rmsnorm_gated(const float* o, const float* w, float eps, void* y, long long n_items, int Dv,
-                                        int dtype, const void* gate, int gate_ld, int items_per_row,
-                                        cudaStream_t stream) {
-  if (n_items < 0 || Dv <= 0 || (gate && (items_per_row <= 0 || gate_ld < items_per_row * Dv))) return LLMIE_ERR_BAD_ARG;
+// gate (of `dtype`, rows gate_ld apart, items_per_row items a row) or null: y is also multiplied by sigmoid(gate), or by
+// silu(gate) with `silu`. w_items > 1: w float32 [w_items, Dv], item i uses row i % w_items.
+extern "C" int llmie_head_rmsnorm_ex(const float* o, const float* w, float eps, void* y, long long n_items, int Dv,
+                                     int dtype, const void* gate, int gate_ld, int items_per_row, int silu, int w_items,
+                                     cudaStream_t stream) {
+  if (n_items < 0 || Dv <= 0 || w_items <= 0 || (gate && (items_per_row <= 0 || gate_ld < items_per_row * Dv))) return LLMIE_ERR_BAD_ARG;
   if (n_items == 0) return LLMIE_OK;
   if (Dv >= 512 && Dv % 4 == 0 && aligned16(o) && aligned16(w) && n_items <= 0x7fffffffLL) {
     // wide items: a block each
     const dim3 grid((unsigned)n_items), block(Dv >= 1024 ? 256 : 128);
     if (dtype == LLMIE_F32)
       launch_k(row_rmsnorm_kernel<float>, grid, block, 0, stream, o, w, eps, (float*)y, Dv, (const float*)gate, gate_ld,
-               items_per_row);
+               items_per_row, silu, w_items);
     else if (dtype == LLMIE_BF16)
       launch_k(row_rmsnorm_kernel<__nv_bfloat16>, grid, block, 0, stream, o, w, eps, (__nv_bfloat16*)y, Dv,
-               (const __nv_bfloat16*)gate, gate_ld, items_per_row);
+               (const __nv_bfloat16*)gate, gate_ld, items_per_row, silu, w_items);
     else
       return LLMIE_ERR_DTYPE;
     LLMIE_LAUNCH_CHECK();
@@ -828,19 +835,25 @@ extern "C" int llmie_head_rmsnorm_gated(const float* o, const float* w, float ep
   const dim3 grid((unsigned)blocks), block(warps * 32);
   if (dtype == LLMIE_F32)
     launch_k(head_rmsnorm_kernel<float>, grid, block, 0, stream, o, w, eps, (float*)y, Dv, (size_t)n_items,
-             (const float*)gate, gate_ld, items_per_row);
+             (const float*)gate, gate_ld, items_per_row, silu, w_items);
   else if (dtype == LLMIE_BF16)
     launch_k(head_rmsnorm_kernel<__nv_bfloat16>, grid, block, 0, stream, o, w, eps, (__nv_bfloat16*)y, Dv,
-             (size_t)n_items, (const __nv_bfloat16*)gate, gate_ld, items_per_row);
+             (size_t)n_items, (const __nv_bfloat16*)gate, gate_ld, items_per_row, silu, w_items);
   else
     return LLMIE_ERR_DTYPE;
   LLMIE_LAUNCH_CHECK();
   return LLMIE_OK;
 }
 
+extern "C" int llmie_head_rmsnorm_gated(const float* o, const float* w, float eps, void* y, long long n_items, int Dv,
+                                        int dtype, const void* gate, int gate_ld, int items_per_row,
+                                        cudaStream_t stream) {
+  return llmie_head_rmsnorm_ex(o, w, eps, y, n_items, Dv, dtype, gate, gate_ld, items_per_row, 0, 1, stream);
+}
+
 extern "C" int llmie_head_rmsnorm(const float* o, const float* w, float eps, void* y, long long n_items, int Dv,
                                   int dtype, cudaStream_t stream) {
-  return llmie_head_rmsnorm_gated(o, w, eps, y, n_items, Dv, dtype, nullptr, 0, 1, stream);
+  return llmie_head_rmsnorm_ex(o, w, eps, y, n_items, Dv, dtype, nullptr, 0, 1, 0, 1, stream);
 }
 
 template <typename TP, typename TO>

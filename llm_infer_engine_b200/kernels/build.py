@@ -33,6 +33,7 @@ FAMILIES: Dict[str, tuple] = {
     "parallel_elementwise": ("parallel_elementwise.cu", [], []),
     "scaled_elementwise": ("scaled_elementwise.cu", [], []),
     "recurrent": ("recurrent.cu", [], []),
+    "matrix_state": ("matrix_state.cu", [], []),
     "ssm": ("ssm.cu", [], []),
     "conv_attention": ("conv_attention.cu", [], []),
     "grouped_gemm": ("grouped_gemm.cu", [], []),

@@ -330,6 +330,7 @@ def _row_slice(t: torch.Tensor, what: str, dtype, rows: int, cols: int) -> int:
 
 
 ACT_NONE, ACT_RELU, ACT_RELU2, ACT_GELU_TANH, ACT_SILU = 0, 1, 2, 3, 4
+GATE_CLAMPED = 5       # a gated pair only: clamped gate and linear part (csrc/common.cuh: gated_pair)
 ACTIVATIONS = {"none": ACT_NONE, "relu": ACT_RELU, "relu2": ACT_RELU2, "gelu_tanh": ACT_GELU_TANH, "silu": ACT_SILU}
 
 
@@ -774,9 +775,10 @@ def gemm_skinny_add_bias(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bi
     return out
 
 
-def gemm_skinny_gated(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: int) -> torch.Tensor:
+def gemm_skinny_gated(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: int, alpha: float = 0.0,
+                      limit: float = 0.0) -> torch.Tensor:
     """out (bfloat16 [batch, N / 2]) = act(x Wg^T) * (x Wu^T) for w = [gate rows; up rows] in one kernel, for a few
-    rows of x; act an ACT_* code."""
+    rows of x; act an ACT_* code or GATE_CLAMPED (see gated_act)."""
     batch, K = x.shape
     N = w.shape[0]
     _need(x, "x", torch.bfloat16)
@@ -785,8 +787,9 @@ def gemm_skinny_gated(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: 
         raise KernelError(f"gemm_skinny_gated: shape batch={batch}, N={N}, K={K} or activation {act} is not supported")
     _need(out, "out", torch.bfloat16, (batch, N // 2))
     _work(_nbytes(x, w, out), 2.0 * batch * N * K)
-    f = _fn("gemm_skinny", "llmie_gemm_skinny_gated", [_c_void_p] * 3 + [_c_int] * 5 + [_c_void_p])
-    _check(f(x.data_ptr(), w.data_ptr(), out.data_ptr(), batch, N, K, N // 2, int(act), _stream()), "gemm_skinny_gated")
+    f = _fn("gemm_skinny", "llmie_gemm_skinny_gated", [_c_void_p] * 3 + [_c_int] * 5 + [_c_float, _c_float, _c_void_p])
+    _check(f(x.data_ptr(), w.data_ptr(), out.data_ptr(), batch, N, K, N // 2, int(act), float(alpha), float(limit),
+             _stream()), "gemm_skinny_gated")
     return out
 
 
@@ -1221,14 +1224,16 @@ def add_dyt(h, d1, d2, alpha, weight, bias, out, rows=None):
     return out
 
 
-def gated_act(gate_up: torch.Tensor, out: torch.Tensor, act: int) -> torch.Tensor:
-    """out[t, j] = act(gate_up[t, j]) * gate_up[t, ff + j]; gate_up [T, 2 ff], out [T, ff]; act an ACT_* code."""
+def gated_act(gate_up: torch.Tensor, out: torch.Tensor, act: int, alpha: float = 0.0, limit: float = 0.0) -> torch.Tensor:
+    """out[t, j] = act(gate_up[t, j]) * gate_up[t, ff + j]; gate_up [T, 2 ff], out [T, ff]; act an ACT_* code. With
+    GATE_CLAMPED, out = g sigmoid(alpha g) (u + 1) with g = min(gate, limit) and u the linear part clamped to +-limit."""
     T, ff = out.shape
     _need(out, "out")
     _need(gate_up, "gate_up", out.dtype, (T, 2 * ff))
     _work(_nbytes(gate_up, out))
-    f = _fn("parallel_elementwise", "llmie_gated_act", [_c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p])
-    _check(f(gate_up.data_ptr(), out.data_ptr(), T, ff, int(act), _dt(out, "out"), _stream()), "gated_act")
+    f = _fn("parallel_elementwise", "llmie_gated_act", [_c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_float,
+                                                        _c_int, _c_void_p])
+    _check(f(gate_up.data_ptr(), out.data_ptr(), T, ff, int(act), float(alpha), float(limit), _dt(out, "out"), _stream()), "gated_act")
     return out
 
 
@@ -1327,17 +1332,19 @@ def routed_gemm_nt(a, a_rows, w, out, out_rows, tile_group, n_positions: int, sm
 
 
 # ------------------------------------------------------------------------------------------ routed feed-forward
-ROUTE_SOFTMAX_TOP, ROUTE_SOFTMAX_ALL, ROUTE_SIGMOID = 0, 1, 2
+ROUTE_SOFTMAX_TOP, ROUTE_SOFTMAX_ALL, ROUTE_SIGMOID, ROUTE_SIGMOID_GROUPS = 0, 1, 2, 3
 
 
-def moe_route(x, w, bias, ids, weights, scores_over_all=False, correction=None, out_scale: float = 1.0):
+def moe_route(x, w, bias, ids, weights, scores_over_all=False, correction=None, out_scale: float = 1.0, groups=(1, 1)):
     """Router of a mixture of experts: logits = x @ w^T + bias in float32; ids int32 [T, top] receive the `top`
     largest (ties: the lower index), weights float32 [T, top] the softmax over those logits alone.
     x [T, d] float32 or bfloat16; w float32 [E, d]; bias float32 [E] or None.
     `scores_over_all`: the scores are the softmax over ALL logits, the choice goes by score + correction (float32 [E]
     or None) and the weights are the chosen scores / (their sum + 1e-20) * out_scale. `scores_over_all` may also be one
     of the ROUTE_* codes; ROUTE_SIGMOID: the `top` largest logits choose and the weights are sigmoid(logit) * out_scale of
-    the chosen ones, not normalised."""
+    the chosen ones, not normalised; ROUTE_SIGMOID_GROUPS: the same weights, chosen by sigmoid(logit) + correction among
+    the experts of the keep best of count equal groups of neighbours (`groups` = (count, keep); a group's score is the sum
+    of its two largest choice scores)."""
     T, d = x.shape
     E = w.shape[0]
     top = ids.shape[1]
@@ -1350,10 +1357,11 @@ def moe_route(x, w, bias, ids, weights, scores_over_all=False, correction=None, 
     if correction is not None:
         _need(correction, "correction", torch.float32, (E,))
     _work(_nbytes(x, w, ids, weights), 2.0 * T * E * d)
-    f = _fn("moe", "llmie_moe_route_ex", [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p] + [_c_int] * 5 +
-            [_c_void_p, _c_float, _c_void_p])
+    f = _fn("moe", "llmie_moe_route_groups", [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p] +
+            [_c_int] * 5 + [_c_void_p, _c_float, _c_int, _c_int, _c_void_p])
     _check(f(x.data_ptr(), _dt(x, "x"), w.data_ptr(), _ptr(bias), ids.data_ptr(), weights.data_ptr(), T, d, E, top,
-             int(scores_over_all), _ptr(correction), float(out_scale), _stream()), "moe_route")
+             int(scores_over_all), _ptr(correction), float(out_scale), int(groups[0]), int(groups[1]), _stream()),
+           "moe_route")
 
 
 def moe_max_tiles(n_pairs: int, n_experts: int, tile: int) -> int:
@@ -1621,6 +1629,43 @@ def scaled_add_rmsnorm(h, d1, c1: float, d2, c2: float, scale, weight, eps: floa
     return out
 
 
+def sandwich_add_norm(h, terms, term_weights, term_eps: float, out_weight, out_eps: float, weight, eps: float, out,
+                      rows=None):
+    """A branch with a norm behind it closes and the norm in front of the next one opens it, N = division by the root mean
+    square over a row: b = sum of c (t or N(t) w_t), h += N(b) out_weight (float32, in place, when rows is None),
+    out = N(h) weight. `terms`: one or two (tensor [T, d], constant); `term_weights`: for each float32 [d] or None; weight
+    and out may both be None (the add alone), or weight alone (out receives the new stream). With `rows` (int32 [n_out])
+    only those rows are produced and h stays as it is."""
+    T, d = h.shape
+    n_out = T if rows is None else rows.shape[0]
+    _need(h, "h", torch.float32)
+    (t1, c1), (t2, c2) = terms[0], (terms[1] if len(terms) > 1 else (None, 0.0))
+    w1, w2 = term_weights[0], (term_weights[1] if len(terms) > 1 else None)
+    for name, t in (("first term", t1), ("second term", t2)):
+        if t is not None:
+            _need(t, name, None, (T, d))
+    for name, t in (("first term's weight", w1), ("second term's weight", w2), ("out_weight", out_weight),
+                    ("weight", weight)):
+        if t is not None:
+            _need(t, name, torch.float32, (d,))
+    if weight is not None and out is None:
+        raise KernelError("sandwich_add_norm: a weight needs an out")
+    if rows is not None:
+        _need(rows, "rows", torch.int32, (n_out,))
+        if n_out == 0:
+            return out
+    out_ld = _row_slice(out, "out", out.dtype, n_out, d) if out is not None else d
+    _work((2 * _nbytes(h) if rows is None else n_out * d * 4) + _nbytes(t1, t2, out))
+    f = _fn("scaled_elementwise", "llmie_sandwich_add_norm",
+            [_c_void_p, _c_void_p, _c_int, _c_float, _c_void_p, _c_void_p, _c_int, _c_float, _c_void_p, _c_float, _c_void_p,
+             _c_float, _c_void_p, _c_float, _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_void_p])
+    _check(f(h.data_ptr(), t1.data_ptr(), _dt(t1, "first term"), float(c1), _ptr(w1), _ptr(t2),
+             _dt(t2, "second term") if t2 is not None else 0, float(c2), _ptr(w2), float(term_eps), out_weight.data_ptr(),
+             float(out_eps), _ptr(weight), float(eps), _ptr(out), int(out_ld), _dt(out, "out") if out is not None else 0,
+             _ptr(rows), n_out, d, _stream()), "sandwich_add_norm")
+    return out
+
+
 def poly_norm(z, coef, eps: float, out):
     """out = a N(z) + b N(z^2) + c N(z^3) + e per row, N(t) = t / sqrt(mean(t^2) + eps); coef float32 [4] = (a, b, c, e)
     on the device; z, out [T, n] of one dtype; float32 arithmetic."""
@@ -1737,23 +1782,26 @@ def _matrix_scan_stepped(q, f, v, v_ld, state, cu_q, seq_slot, out, ws, decay, n
            "matrix_scan_stepped")
 
 
-def head_rmsnorm(o, weight, eps: float, out, vdim: int, gate=None):
+def head_rmsnorm(o, weight, eps: float, out, vdim: int, gate=None, gate_silu: bool = False):
     """out = o / sqrt(mean(o^2) + eps) * weight over every run of vdim columns (a head; vdim = the row's width: the
-    concatenated heads together, with a weight per column); o float32 [T, heads vdim]; weight float32 [vdim]; out of
-    the activation type. `gate` ([T, heads vdim] of out's type, possibly a column slice): out is also multiplied by
-    sigmoid(gate)."""
+    concatenated heads together, with a weight per column); o float32 [T, heads vdim]; weight float32 [vdim], shared by
+    the heads, or [heads vdim]; out of the activation type. `gate` ([T, heads vdim] of out's type, possibly a column
+    slice): out is also multiplied by sigmoid(gate), or by silu(gate) with `gate_silu`."""
     T, n = o.shape
     _need(o, "o", torch.float32)
-    _need(weight, "weight", torch.float32, (vdim,))
-    _need(out, "out", None, (T, n))
     if n % vdim:
         raise KernelError("head_rmsnorm: the row is not a whole number of heads")
+    w_items = weight.shape[0] // vdim
+    if w_items not in (1, n // vdim):
+        raise KernelError(f"head_rmsnorm: {weight.shape[0]} weights for {n // vdim} heads of {vdim}")
+    _need(weight, "weight", torch.float32, (w_items * vdim,))
+    _need(out, "out", None, (T, n))
     gate_ld = _row_slice(gate, "gate", out.dtype, T, n) if gate is not None else 0
     _work(_nbytes(o, out) + (T * n * out.element_size() if gate is not None else 0))
-    f = _fn("recurrent", "llmie_head_rmsnorm_gated", [_c_void_p, _c_void_p, _c_float, _c_void_p, ctypes.c_longlong, _c_int,
-                                                      _c_int, _c_void_p, _c_int, _c_int, _c_void_p])
+    f = _fn("recurrent", "llmie_head_rmsnorm_ex", [_c_void_p, _c_void_p, _c_float, _c_void_p, ctypes.c_longlong, _c_int,
+                                                   _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p])
     _check(f(o.data_ptr(), weight.data_ptr(), float(eps), out.data_ptr(), T * (n // vdim), vdim, _dt(out, "out"),
-             _ptr(gate), gate_ld, n // vdim, _stream()), "head_rmsnorm")
+             _ptr(gate), gate_ld, n // vdim, 1 if gate_silu else 0, w_items, _stream()), "head_rmsnorm")
     return out
 
 
@@ -2002,4 +2050,169 @@ def unit_scan(gates, proj, y_off: int, x_off: int, y_bias, x_bias, act: int, sta
              int(act), state.data_ptr(), conv_state.data_ptr(), cu_q.data_ptr(), seq_slot.data_ptr(), out.data_ptr(),
              n_seqs, C, int(block_width), K, 1 if write_state else 0, 1 if max_len > UNIT_CHUNKS else 0,
              _dt(proj, "proj"), _stream()), "unit_scan")
+    return out
+
+
+# ------------------------------------------------------------------------------------------ matrix states by channel
+FORM_KEY_DECAY, FORM_BONUS, FORM_DELTA = 0, 1, 2      # csrc/matrix_state.cu
+GATE_POWER, GATE_DOUBLE_EXP = 0, 1                     # sigmoid(z)^(1/tau); exp(-exp(z)) with tanh in front of the product
+MAX_CHANNEL_DIM, MAX_GATE_RANK = 512, 512
+
+
+def low_rank_gate(x, Bt, bias, out, mode: int, tau: float = 1.0):
+    """out[t, c] = f(bias[c] + sum_r Bt[r, c] g(x[t, r])): the decay of every key channel from a few numbers per token.
+    GATE_POWER: f = sigmoid^(1/tau), g = identity; GATE_DOUBLE_EXP: f = exp(-exp(.)), g = tanh. x [T, R] float32 or
+    bfloat16, possibly a column slice; Bt float32 [R, N]; out float32 [T, N]."""
+    T, R = x.shape
+    N = Bt.shape[1]
+    ld = _row_slice(x, "x", x.dtype, T, R)
+    _need(Bt, "Bt", torch.float32, (R, N))
+    _need(bias, "bias", torch.float32, (N,))
+    _need(out, "out", torch.float32, (T, N))
+    _work(_nbytes(Bt, out) + T * R * x.element_size(), 2.0 * T * R * N)
+    f = _fn("matrix_state", "llmie_low_rank_gate",
+            [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p] + [_c_int] * 4 + [_c_float, _c_int, _c_void_p])
+    _check(f(x.data_ptr(), ld, Bt.data_ptr(), bias.data_ptr(), out.data_ptr(), R, N, T, int(mode), 1.0 / tau,
+             _dt(x, "x"), _stream()), "low_rank_gate")
+    return out
+
+
+def delta_prepare(qkv, ba, b_off: int, a_off: int, A, dt_bias, eps: float, q_scale: float, qn, kn, scal, qk, heads: int,
+                  groups: int, dim: int):
+    """What the delta rule reads: unit vectors of the `groups` heads of q and k at the start of qkv's rows (x / sqrt(sum
+    x^2 + eps), q also times q_scale) -> qn, kn float32 [T, groups dim]; q . k -> qk float32 [T, groups]; scal float32
+    [T, heads, 2] = (sigmoid(b), exp(-A softplus(a + dt_bias))) from the columns b_off and a_off of ba [T, ...]."""
+    T = qkv.shape[0]
+    _need(qkv, "qkv")
+    _need(ba, "ba", None, (T, None))
+    for name, t, shape in (("A", A, (heads,)), ("dt_bias", dt_bias, (heads,)), ("qn", qn, (T, groups * dim)),
+                           ("kn", kn, (T, groups * dim)), ("scal", scal, (T, heads, 2)), ("qk", qk, (T, groups))):
+        _need(t, name, torch.float32, shape)
+    _work(2 * T * groups * dim * (qkv.element_size() + 4) + _nbytes(scal, qk))
+    f = _fn("matrix_state", "llmie_delta_prepare",
+            [_c_void_p, _c_int, _c_int, _c_void_p] + [_c_int] * 4 + [_c_void_p, _c_void_p, _c_float, _c_float] +
+            [_c_void_p] * 4 + [_c_int] * 4 + [_c_void_p])
+    _check(f(qkv.data_ptr(), qkv.shape[1], _dt(qkv, "qkv"), ba.data_ptr(), ba.shape[1], int(b_off), int(a_off),
+             _dt(ba, "ba"), A.data_ptr(), dt_bias.data_ptr(), float(eps), float(q_scale), qn.data_ptr(), kn.data_ptr(),
+             scal.data_ptr(), qk.data_ptr(), T, heads, groups, dim, _stream()), "delta_prepare")
+
+
+def shift_mix(x, prev, mu, cu_q, tok_seq, seq_slot, out, single: bool = False):
+    """out[s, t] = x[t] + (x_prev - x[t]) mu[s], x_prev the previous token's x (of the slot's `prev`, float32 [slots, 1, d],
+    for a piece's first token). x [T, d]; mu float32 [n, d]; out [n, T, d] of x's type. `single`: every sequence brings
+    one token, and prev is written too (`conv_state_store` does it for other steps)."""
+    T, d = x.shape
+    n = mu.shape[0]
+    _need(x, "x")
+    _need(prev, "prev", torch.float32, (None, 1, d))
+    _need(mu, "mu", torch.float32, (n, d))
+    _need(out, "out", x.dtype, (n, T, d))
+    for name, t in (("cu_q", cu_q), ("tok_seq", tok_seq), ("seq_slot", seq_slot)):
+        _need(t, name, torch.int32)
+    _work(_nbytes(x, out))
+    f = _fn("matrix_state", "llmie_shift_mix", [_c_void_p] * 7 + [_c_int] * 5 + [_c_void_p])
+    _check(f(x.data_ptr(), prev.data_ptr(), mu.data_ptr(), cu_q.data_ptr(), tok_seq.data_ptr(), seq_slot.data_ptr(),
+             out.data_ptr(), n, d, T, 1 if single else 0, _dt(x, "x"), _stream()), "shift_mix")
+    return out
+
+
+def channel_scan(form: int, q, k, v, state, cu_q, seq_slot, out, n_seqs: int, heads: int, groups: int, dim: int, vdim: int,
+                 q_scale: float = 1.0, gate=None, bonus=None, scal=None, qk=None):
+    """The recurrences of csrc/matrix_state.cu over pieces of any length. q, k [T, groups dim] of one type and v
+    [T, heads vdim] (column slices allowed); state float32 [slots, heads, dim, vdim] is read and written; out float32
+    [T, heads vdim]. FORM_KEY_DECAY, FORM_BONUS: gate float32 [T, groups dim] (and bonus float32 [groups dim]);
+    FORM_DELTA: scal, qk of `delta_prepare`."""
+    T = q.shape[0]
+    q_ld, k_ld = _row_slice(q, "q", q.dtype, T, groups * dim), _row_slice(k, "k", q.dtype, T, groups * dim)
+    v_ld = _row_slice(v, "v", v.dtype, T, heads * vdim)
+    _need(state, "state", torch.float32, (None, heads, dim, vdim))
+    _need(out, "out", torch.float32, (T, heads * vdim))
+    _need(cu_q, "cu_q", torch.int32)
+    _need(seq_slot, "seq_slot", torch.int32)
+    for name, t, shape in (("gate", gate, (T, groups * dim)), ("bonus", bonus, (groups * dim,)),
+                           ("scal", scal, (T, heads, 2)), ("qk", qk, (T, groups))):
+        if t is not None:
+            _need(t, name, torch.float32, shape)
+    _work(2 * T * groups * dim * q.element_size() + T * heads * vdim * v.element_size() + _nbytes(gate, scal, qk, out) +
+          8.0 * n_seqs * heads * dim * vdim, (8.0 if form == FORM_DELTA else 5.0) * T * heads * dim * vdim)
+    f = _fn("matrix_state", "llmie_channel_scan",
+            [_c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_float, _c_void_p, _c_int, _c_int] + [_c_void_p] * 8 +
+            [_c_int] * 6 + [_c_void_p])
+    _check(f(q.data_ptr(), q_ld, k.data_ptr(), k_ld, _dt(q, "q"), float(q_scale), v.data_ptr(), v_ld, _dt(v, "v"),
+             _ptr(gate), _ptr(bonus), _ptr(scal), _ptr(qk), state.data_ptr(), cu_q.data_ptr(), seq_slot.data_ptr(),
+             out.data_ptr(), n_seqs, heads, groups, dim, vdim, int(form), _stream()), "channel_scan")
+    return out
+
+
+def state_step_supported(dim: int, vdim: int) -> bool:
+    """Whether the one-token kernel takes a state of [dim, vdim] per head."""
+    return bool(_fn("matrix_state", "llmie_state_step_ok", [_c_int, _c_int], query=True)(dim, vdim))
+
+
+def state_step(form: int, q, k, v, state, cu_q, seq_slot, out, n_seqs: int, heads: int, groups: int, dim: int, vdim: int,
+               norm_w, norm_eps: float, z, q_scale: float = 1.0, bonus=None, x=None, Bt=None, gate_bias=None,
+               gate_mode: int = 0, tau: float = 1.0, ba=None, b_off: int = 0, a_off: int = 0, A=None, dt_bias=None,
+               unit_eps: float = 0.0):
+    """One token per sequence through the same recurrences, with what surrounds them in the same kernel: decays from x
+    (as `low_rank_gate`; FORM_KEY_DECAY, FORM_BONUS) or unit vectors, rate and decay (as `delta_prepare`; FORM_DELTA, q, k,
+    v float32), then out = o / sqrt(mean(o^2) + norm_eps) norm_w silu(z) per head. norm_w float32 [vdim], shared by the
+    heads, or [heads vdim]; z, out [T, heads vdim] of the activation type (z possibly a column slice)."""
+    T = q.shape[0]
+    q_ld, k_ld = _row_slice(q, "q", q.dtype, T, groups * dim), _row_slice(k, "k", q.dtype, T, groups * dim)
+    v_ld, z_ld = _row_slice(v, "v", q.dtype, T, heads * vdim), _row_slice(z, "z", out.dtype, T, heads * vdim)
+    _need(state, "state", torch.float32, (None, heads, dim, vdim))
+    _need(out, "out", None, (T, heads * vdim))
+    _need(cu_q, "cu_q", torch.int32)
+    _need(seq_slot, "seq_slot", torch.int32)
+    shared = norm_w.shape[0] == vdim
+    _need(norm_w, "norm_w", torch.float32, (vdim if shared else heads * vdim,))
+    R, x_ld = 0, 0
+    if form != FORM_DELTA:
+        R = x.shape[1]
+        x_ld = _row_slice(x, "x", x.dtype, T, R)
+        _need(Bt, "Bt", torch.float32, (R, groups * dim))
+        _need(gate_bias, "gate_bias", torch.float32, (groups * dim,))
+        if form == FORM_BONUS:
+            _need(bonus, "bonus", torch.float32, (groups * dim,))
+    else:
+        _need(ba, "ba", out.dtype, (T, None))
+        _need(A, "A", torch.float32, (heads,))
+        _need(dt_bias, "dt_bias", torch.float32, (heads,))
+    _work(8.0 * n_seqs * heads * dim * vdim + _nbytes(Bt, out) + T * heads * vdim * (q.element_size() + out.element_size()),
+          (8.0 if form == FORM_DELTA else 5.0) * T * heads * dim * vdim)
+    f = _fn("matrix_state", "llmie_state_step",
+            [_c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_float, _c_void_p, _c_int] + [_c_void_p] * 4 +
+            [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_float] +
+            [_c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_float] +
+            [_c_void_p, _c_int, _c_float, _c_void_p, _c_int, _c_void_p] + [_c_int] * 7 + [_c_void_p])
+    _check(f(q.data_ptr(), q_ld, k.data_ptr(), k_ld, _dt(q, "q"), float(q_scale), v.data_ptr(), v_ld, _ptr(bonus),
+             state.data_ptr(), cu_q.data_ptr(), seq_slot.data_ptr(),
+             _ptr(x), x_ld, _dt(x, "x") if x is not None else 0, _ptr(Bt), _ptr(gate_bias), R, int(gate_mode), 1.0 / tau,
+             _ptr(ba), ba.shape[1] if ba is not None else 0, int(b_off), int(a_off), _ptr(A), _ptr(dt_bias),
+             float(unit_eps), norm_w.data_ptr(), 0 if shared else vdim, float(norm_eps), z.data_ptr(), z_ld,
+             out.data_ptr(), _dt(out, "out"), n_seqs, heads, groups, dim, vdim, int(form), _stream()), "state_step")
+    return out
+
+
+STACKED_BEST_ROWS = 16     # up to here this library's kernel, above it the library's batched GEMM
+
+
+def stacked_gemm_nt(a, w, out):
+    """out[g] = a[g] @ w[g]^T for a few products of one shape with inputs of their own: a [G, T, K], w [G, N, K], out
+    [G, T, N]. bfloat16 with more rows than one-token steps bring: the library's batched GEMM, as single products go to
+    its plain one; otherwise this library's grouped kernel (float32: true 32-bit, fixed order of k)."""
+    G, T, K = a.shape
+    N = w.shape[1]
+    _need(a, "a")
+    _need(w, "w", a.dtype, (G, N, K))
+    _need(out, "out", None, (G, T, N))
+    _work(_nbytes(a, w, out), 2.0 * G * T * N * K)
+    if a.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and T > STACKED_BEST_ROWS:
+        def run():
+            return torch.bmm(a, w.transpose(1, 2), out=out)
+        t = trace.timer
+        return run() if t is None else t.run("library_bmm", run, ())
+    f = _fn("grouped_gemm", "llmie_grouped_gemm_nt", _GROUPED_ARGS)
+    _check(f(a.data_ptr(), K, T * K, None, w.data_ptr(), N * K, K, out.data_ptr(), N, T * N, None, None, 0, G, T, N, K, 0, 0,
+             1 if T <= GROUPED_SMALL_ROWS else 0, _dt(a, "a"), _dt(out, "out"), _stream()), "stacked_gemm_nt")
     return out

@@ -136,28 +136,51 @@ class ScaledDelta:
     (the bias of a branch's last product) or None. A mixer made of two
     mixers returns one without a vector; a block with a learned scale per channel puts its vector on whatever its
     branch returned. A norm whose kernel knows the form adds it while it reads the stream; `materialize()` gives the
-    plain float32 tensor to everything else."""
+    plain float32 tensor to everything else.
 
-    def __init__(self, terms, vector: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None):
+    Norms on the way, N being the division by the root mean square over a row: `term_norms` = (a float32 [d] weight per
+    term, eps) makes each term N(t) w before its constant; `out_norm` = (float32 [d] weight, eps) makes the whole sum
+    N(sum) w (a block with a norm behind its branches). Neither goes with a vector or a bias."""
+
+    def __init__(self, terms, vector: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None,
+                 term_norms=None, out_norm=None):
         terms = [(t, float(c)) for t, c in terms]
         if not 1 <= len(terms) <= 2:
             raise ValueError("a ScaledDelta has one or two terms")
+        if (term_norms or out_norm) and (vector is not None or bias is not None):
+            raise ValueError("norms on a branch output do not go with a vector or a bias")
         self.terms, self.vector, self.bias = terms, vector, bias
+        self.term_norms, self.out_norm = term_norms, out_norm
 
     @staticmethod
     def of(y, vector: Optional[torch.Tensor]) -> "ScaledDelta":
         """`y` (a tensor or a ScaledDelta without a vector) times `vector`, channel by channel."""
         if isinstance(y, ScaledDelta):
-            if y.vector is not None:
-                raise ValueError("this branch output already carries a vector")
+            if y.vector is not None or y.term_norms or y.out_norm:
+                raise ValueError("this branch output already carries a vector or norms")
             return ScaledDelta(y.terms, vector, None if y.bias is None else (y.bias * vector).contiguous())
         return ScaledDelta([(y, 1.0)], vector)
+
+    @staticmethod
+    def normed(y, weight: torch.Tensor, eps: float) -> "ScaledDelta":
+        """N(y) weight for a branch output `y` (a tensor, or a ScaledDelta without a vector, a bias or such a norm)."""
+        if isinstance(y, ScaledDelta):
+            if y.vector is not None or y.bias is not None or y.out_norm:
+                y = ScaledDelta([(y.materialize(), 1.0)])
+            return ScaledDelta(y.terms, term_norms=y.term_norms, out_norm=(weight, eps))
+        return ScaledDelta([(y, 1.0)], out_norm=(weight, eps))
 
     def add_into(self, h: torch.Tensor, out: Optional[torch.Tensor] = None, weight: Optional[torch.Tensor] = None,
                  eps: float = 0.0, rows: Optional[torch.Tensor] = None) -> None:
         """h (float32 [T, d]) += this, in place; `out`, if given, receives the new rows normed with `weight`, or as they
         are without one. With `rows` only those rows are produced and h is untouched."""
         from ..kernels import ops
+        if self.out_norm:
+            weights, term_eps = self.term_norms or ((None, None), 0.0)
+            ops.sandwich_add_norm(h, self.terms, weights, term_eps, *self.out_norm, weight, eps, out, rows)
+            return
+        if self.term_norms:
+            raise ValueError("terms with norms are added behind a norm over their sum only")
         (t1, c1), (t2, c2) = self.terms[0], (self.terms[1] if len(self.terms) > 1 else (None, 0.0))
         ops.scaled_add_rmsnorm(h, t1, c1, t2, c2, self.vector, weight, eps, out, rows, bias=self.bias)
 

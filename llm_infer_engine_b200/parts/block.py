@@ -290,3 +290,43 @@ class PostNormScaledMixerBlock(PostNormScaledBlock):
 
 register_block("post_norm_scaled", PostNormScaledBlock)
 register_block("post_norm_scaled_mixer", PostNormScaledMixerBlock)
+
+
+class SandwichBlock(Block):
+    """h += out1(mixer(in1(h))); h += out2(feed_forward(in2(h))): a norm in front of each branch and one behind it. The
+    branch's output travels on as a `ScaledDelta` with the norm behind it, and the kernel of the next norm in front of a
+    branch does both norms and the add in one pass over the rows. A constant on what a branch adds belongs to the norm
+    behind it (`output_scale`)."""
+    ROLES = {"mixer": "mixer", "feed_forward": "feed_forward", "mixer_norm": "norm", "feed_forward_norm": "norm",
+             "mixer_out_norm": "norm", "feed_forward_out_norm": "norm"}
+
+    def forward(self, h, pending, ctx, unit, owns_cache):
+        tracing = trace.active()
+        if tracing:
+            trace.push(f"Attn_{ctx.entry}")
+        x = self.mixer_norm.forward(h, pending)
+        n = self.mixer_out_norm
+        mixed = ScaledDelta.normed(call_branch(self.mixer, x, ctx, unit, owns_cache), n.weight, n.eps)
+        if tracing:
+            trace.pop()
+            trace.push(f"FFN_{ctx.entry}")
+        x = self.feed_forward_norm.forward(h, mixed)
+        n = self.feed_forward_out_norm
+        out = ScaledDelta.normed(call_branch(self.feed_forward, x, ctx), n.weight, n.eps)
+        if tracing:
+            trace.pop()
+        return h, out
+
+
+class SandwichMixerBlock(Block):
+    """The same arrangement for a layer without a feed-forward: h += out1(mixer(in1(h)))."""
+    ROLES = {"mixer": "mixer", "mixer_norm": "norm", "mixer_out_norm": "norm"}
+
+    def forward(self, h, pending, ctx, unit, owns_cache):
+        x = self.mixer_norm.forward(h, pending)
+        n = self.mixer_out_norm
+        return h, ScaledDelta.normed(call_branch(self.mixer, x, ctx, unit, owns_cache), n.weight, n.eps)
+
+
+register_block("sandwich", SandwichBlock)
+register_block("sandwich_mixer", SandwichMixerBlock)

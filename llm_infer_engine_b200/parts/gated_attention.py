@@ -46,7 +46,7 @@ import torch
 from ..cache.cache import KVRequest
 from ..kernels import ops, trace
 from .base import AttentionOptions, DeferredBranchAdd, Mixer, ParamSpec, build_part, register_mixer
-from .linear import Linear
+from .linear import Linear, pad_rows
 
 _DEFAULT_NAMES = {"q": "q", "k": "k", "v": "v", "gate": "g", "o": "o", "q_norm": "q.norm", "k_norm": "k.norm",
                   "blend": "vmix", "distance_bias": "rel", "sink": "sink", "sigmoid_bias": "pb"}
@@ -160,7 +160,8 @@ class GatedAttention(Mixer):
         n = self.names
         ws = [tensors[n["q"]], tensors[n["k"]], tensors[n["v"]]] + ([tensors[n["gate"]]] if self.gate else [])
         dtype = torch.float32 if any(w.dtype == torch.float32 for w in ws) else ws[0].dtype
-        self.proj = Linear(torch.cat([w.to(dtype) for w in ws], dim=0))
+        packed = torch.cat([w.to(dtype) for w in ws], dim=0)
+        self.proj = Linear(pad_rows(packed) if self.head_gate else packed)     # a gate per head: rows of any number
         self.o = Linear(tensors[n["o"]])
         if self.qk_norm_eps is not None:
             self.q_w = tensors[n["q_norm"]].to(torch.float32).contiguous()
@@ -226,7 +227,8 @@ class GatedAttention(Mixer):
                               temp_coef=self.temp_coef, temp_every=self.temp_every)
         trace.pop()
         out = torch.empty((T, self.no), dtype=proj.dtype, device=proj.device)
-        gate = proj[:, self.nq + self.nk + self.nv:] if self.gate else None
+        n_qkv = self.nq + self.nk + self.nv
+        gate = proj[:, n_qkv:n_qkv + (self.n_heads if self.head_gate else self.no)] if self.gate else None
         trace.push("FlashDecode" if ctx.decode else "FlashAttn")
         ctx.attention(q, kv, out, self.n_heads, self.n_kv_heads, self.head_dim, self.options,
                       gate=None if self.head_gate else gate)

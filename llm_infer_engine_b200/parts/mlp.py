@@ -15,7 +15,9 @@ from .linear import Linear
 class SwiGLU(FeedForward):
     """params: hidden, intermediate; activation (on the gate: "silu", the default, or any of ops.ACTIVATIONS, e.g.
     "gelu_tanh"); names (checkpoint sub-names of gate, up, down); out_float32 (the branch output is float32 instead
-    of the activations' type: for designs that round nothing between the last product and the residual sum)."""
+    of the activations' type: for designs that round nothing between the last product and the residual sum);
+    activation "clamped": down(g sigmoid(alpha g) (u + 1)) with g = min(gate x, limit) and u = up x clamped to +-limit,
+    with the params gate_alpha and gate_limit."""
 
     adds_to_residual = True
     accepts_deferred_norm = True
@@ -25,9 +27,14 @@ class SwiGLU(FeedForward):
         self.hidden = int(params["hidden"])
         self.intermediate = int(params["intermediate"])
         name = str(params.get("activation", "silu"))
-        if name not in ops.ACTIVATIONS or name == "none":
-            raise ValueError(f"activation {name!r} is not known ({sorted(ops.ACTIVATIONS)})")
-        self.activation = ops.ACTIVATIONS[name]
+        self.gate_alpha = self.gate_limit = 0.0
+        if name == "clamped":
+            self.activation = ops.GATE_CLAMPED
+            self.gate_alpha, self.gate_limit = float(params["gate_alpha"]), float(params["gate_limit"])
+        elif name not in ops.ACTIVATIONS or name == "none":
+            raise ValueError(f"activation {name!r} is not known ({sorted(ops.ACTIVATIONS) + ['clamped']})")
+        else:
+            self.activation = ops.ACTIVATIONS[name]
         self.names = dict({"gate": "gate_proj.weight", "up": "up_proj.weight", "down": "down_proj.weight"},
                           **(params.get("names") or {}))
         self.out_float32 = bool(params.get("out_float32", False))
@@ -68,14 +75,15 @@ class SwiGLU(FeedForward):
             else:
                 x = x.apply()
         if act is None:                              # product, activation and gate in one kernel
-            act = self.gate_up.swiglu(x) if self.activation == ops.ACT_SILU else self.gate_up.gated(x, self.activation)
+            act = self.gate_up.swiglu(x) if self.activation == ops.ACT_SILU else \
+                self.gate_up.gated(x, self.activation, self.gate_alpha, self.gate_limit)
         if act is None:
             gu = self.gate_up(x)
             act = torch.empty((x.shape[0], self.intermediate), dtype=gu.dtype, device=x.device)
             if self.activation == ops.ACT_SILU:
                 ops.swiglu(gu, act)
             else:
-                ops.gated_act(gu, act, self.activation)
+                ops.gated_act(gu, act, self.activation, self.gate_alpha, self.gate_limit)
         if residual is not None and self.down.add_into(act, residual):
             return None
         return self.down(act, out_dtype=torch.float32) if self.out_float32 else self.down(act)

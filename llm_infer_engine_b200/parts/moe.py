@@ -16,7 +16,9 @@ Options: `gated` False makes an expert down_e(act(up_e u)), one product in front
 "softmax_all" is a second rule for the router: s = softmax(z) over ALL its outputs, the `top` largest of s + c are chosen
 (c a stored correction that steers the choice only), and a_t,e = s_t,e / (sum of the chosen s + 1e-20) * `weight_scale`.
 "sigmoid" is a third: s = sigmoid(z) one by one, the `top` largest choose and weigh as they are (times `weight_scale`),
-not normalised. `weight_on` "input" (default "output"): the weight multiplies what the expert READS, y_t = sum over e of
+not normalised. "sigmoid_groups" is a fourth: the same scores weigh, the `top` largest of s + c choose (c as in the second
+rule), and only among the experts of the `groups_keep` best of `groups` equal runs of neighbours, a group's score being the
+sum of its two largest s + c. `weight_on` "input" (default "output"): the weight multiplies what the expert READS, y_t = sum over e of
 expert_e(a_t,e u_t), which is not the same thing under a non-linear expert; the rows are scaled while they are gathered
 into the order of their experts, and the combine adds with weight one.
 `identity_experts` n: the router has n more outputs than there are experts; the last n stand for experts that return
@@ -38,7 +40,8 @@ from ..config.spec import PartSpec
 class RoutedExperts(FeedForward):
     """params: hidden, n_experts, top, expert_ff, activation (default "silu"), router_bias (bool, default True),
     shared_ff (width of the shared expert, None = none), shared_activation (default: `activation`), gated (default
-    True), scoring ("softmax_top", the default, "softmax_all" or "sigmoid"), weight_scale (default 1), weight_on
+    True), scoring ("softmax_top", the default, "softmax_all", "sigmoid" or "sigmoid_groups", which takes groups and
+    groups_keep), weight_scale (default 1), weight_on
     ("output", the default, or "input"), identity_experts (default 0), names (checkpoint sub-names: router, router_bias, correction, expert (a pattern with {e}), gate, up, down,
     shared)."""
 
@@ -56,10 +59,13 @@ class RoutedExperts(FeedForward):
         self.router_bias = bool(p.get("router_bias", True))
         self.gated = bool(p.get("gated", True))
         self.scoring = str(p.get("scoring", "softmax_top"))
-        if self.scoring not in ("softmax_top", "softmax_all", "sigmoid"):
-            raise ValueError(f"scoring must be 'softmax_top', 'softmax_all' or 'sigmoid', got {self.scoring!r}")
+        if self.scoring not in ("softmax_top", "softmax_all", "sigmoid", "sigmoid_groups"):
+            raise ValueError("scoring must be 'softmax_top', 'softmax_all', 'sigmoid' or 'sigmoid_groups', got "
+                             f"{self.scoring!r}")
         self.route_mode = {"softmax_top": ops.ROUTE_SOFTMAX_TOP, "softmax_all": ops.ROUTE_SOFTMAX_ALL,
-                           "sigmoid": ops.ROUTE_SIGMOID}[self.scoring]
+                           "sigmoid": ops.ROUTE_SIGMOID, "sigmoid_groups": ops.ROUTE_SIGMOID_GROUPS}[self.scoring]
+        self.has_correction = self.scoring in ("softmax_all", "sigmoid_groups")
+        self.groups = (1, 1)
         self.weight_on_input = str(p.get("weight_on", "output")) == "input"
         if p.get("weight_on", "output") not in ("output", "input"):
             raise ValueError(f"weight_on must be 'output' or 'input', got {p.get('weight_on')!r}")
@@ -70,6 +76,11 @@ class RoutedExperts(FeedForward):
         self.n_outputs = self.n_experts + self.n_identity          # what the router has outputs for
         if self.top > self.n_outputs or self.n_identity < 0:
             raise ValueError(f"top ({self.top}) must not exceed the router's {self.n_outputs} outputs")
+        if self.scoring == "sigmoid_groups":
+            count, keep = int(p["groups"]), int(p["groups_keep"])
+            if count <= 0 or self.n_outputs % count or not 0 < keep <= count or self.top > self.n_outputs // count * keep:
+                raise ValueError(f"{self.top} of {self.n_outputs} outputs cannot be chosen from {keep} of {count} groups")
+            self.groups = (count, keep)
         self.names = dict({"router": "router", "router_bias": "router.b", "correction": "correction", "expert": "e{e}",
                            "gate": "gate", "up": "up", "down": "down", "shared": "shared"}, **(p.get("names") or {}))
         self.shared = None
@@ -90,7 +101,7 @@ class RoutedExperts(FeedForward):
         specs = {n["router"]: ParamSpec((self.n_outputs, d))}
         if self.router_bias:
             specs[n["router_bias"]] = ParamSpec((self.n_outputs,), role="vector", init=("normal",))
-        if self.scoring == "softmax_all":
+        if self.has_correction:
             specs[n["correction"]] = ParamSpec((self.n_outputs,), role="vector", init=("uniform", -0.05, 0.05))
         for e in range(self.n_experts):
             if self.gated:
@@ -106,7 +117,7 @@ class RoutedExperts(FeedForward):
         n = self.names
         self.w_router = tensors[n["router"]].to(torch.float32).contiguous()
         self.b_router = tensors[n["router_bias"]].to(torch.float32).contiguous() if self.router_bias else None
-        if self.scoring == "softmax_all":
+        if self.has_correction:
             self.correction = tensors[n["correction"]].to(torch.float32).contiguous()
         gu, dn = [], []
         for e in range(self.n_experts):
@@ -135,7 +146,7 @@ class RoutedExperts(FeedForward):
             ids = torch.empty((T, top), dtype=torch.int32, device=dev)
             weights = torch.empty((T, top), dtype=torch.float32, device=dev)
             ops.moe_route(x, self.w_router, self.b_router, ids, weights, self.route_mode, self.correction,
-                          self.weight_scale)
+                          self.weight_scale, self.groups)
             n_pairs = T * top
             small = n_pairs <= ops.GROUPED_SMALL_ROWS
             tile = ops.grouped_tile_rows(small)

@@ -18,7 +18,8 @@ class RMSNorm(Norm):
     """params: size (width of a row), eps; weight_name (the tensor's name under the part's checkpoint name,
     default "weight"; "" = the part's name itself); weight_offset (default 0: the norm multiplies by
     weight_offset + the stored tensor, for checkpoints that store the weight around zero); residual_scale (default 1:
-    the constant alpha of `norm_sum`, the form for blocks whose norm comes AFTER the residual sum)."""
+    the constant alpha of `norm_sum`, the form for blocks whose norm comes AFTER the residual sum); output_scale (default
+    1: a constant on the norm's result, folded into the weight)."""
 
     kind = "rmsnorm"
 
@@ -29,6 +30,7 @@ class RMSNorm(Norm):
         self.weight_name = str(params.get("weight_name", "weight"))
         self.weight_offset = float(params.get("weight_offset", 0.0))
         self.residual_scale = float(params.get("residual_scale", 1.0))
+        self.output_scale = float(params.get("output_scale", 1.0))
         self.weight: Optional[torch.Tensor] = None
 
     def param_specs(self) -> Dict[str, ParamSpec]:
@@ -39,6 +41,8 @@ class RMSNorm(Norm):
         self.weight = tensors[self.weight_name].to(torch.float32).contiguous()   # bf16 -> f32 is exact
         if self.weight_offset:
             self.weight = (self.weight + self.weight_offset).contiguous()        # the sum in float32
+        if self.output_scale != 1.0:
+            self.weight = (self.weight * self.output_scale).contiguous()
 
     def weight_bytes(self) -> int:
         return self.size * 4

@@ -497,6 +497,29 @@ def rogizen_config(width: int, heads: int, kv_heads: int, head_dim: int, ff: int
             "layers": layers}
 
 
+def selinex_config(width: int, heads: int, kv_heads: int, head_dim: int, ff: int, vocab: int, n_layers: int,
+                   window: int) -> dict:
+    """A Selinex configuration with a Llama shape's layer sizes. Layers cycle through four kinds: window attention with a
+    gate per head beside gated linear attention (as many heads, half a head size of key channels and a head size of value
+    channels) + dense feed-forward, rotated window attention beside time mixing (as many heads of a head size) + routed
+    experts, the gated delta rule (as many heads, a head size of key and of value channels, 4 taps) + routed experts, the
+    first pair again + routed experts. The routed feed-forward uses 4 of 16 experts of ff / 4, from two of four groups (the
+    active width of the dense one). The loop holds all layers and runs once, so that as many layers run as in the other
+    design."""
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5,
+            "mask": {"size": window} if window else None}
+    first = {"left": left, "right": {"heads": heads, "dim": head_dim // 2, "vdim": head_dim, "tau": 16.0},
+             "left_scale": 0.5, "right_scale": 0.5}
+    second = {"left": dict(left, rot={"base": 10000.0, "dims": head_dim}), "right": {"heads": heads, "dim": head_dim}}
+    delta = {"heads": heads, "kv_heads": heads, "dim": head_dim, "vdim": head_dim, "conv": 4}
+    dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+    moe = {"kind": "moe", "router": {"experts": 16, "top": 4, "groups": {"count": 4, "keep": 2}}, "expert": {"ff": ff // 4}}
+    kinds = [("parallel", first, dense), ("parallel_2", second, moe), ("delta", delta, moe), ("parallel", first, moe)]
+    layers = [{"type": k, "mixer": json.loads(json.dumps(m)), "mlp": f} for k, m, f in (kinds[i % 4] for i in range(n_layers))]
+    return {"architecture": "Selinex", "vocab": vocab, "width": width, "residual_mult": 0.5, "norm": {"eps": 1e-6},
+            "loop": {"start": 0, "stop": n_layers, "times": 1}, "layers": layers}
+
+
 def step_tables(engine, pk: dict, title: str, batch: int = 8) -> str:
     """Per-kernel tables (eager steps, CUDA events) of a decode step at `batch` sequences and of a 2,048-token
     prompt."""
@@ -536,8 +559,8 @@ def step_tables(engine, pk: dict, title: str, batch: int = 8) -> str:
 
 def run_designs(args, pk: dict, which: str = "Zemivik") -> str:
     """Zemivik (or, with which="Dofipel", Dofipel with a window of 1,024) beside Llama at equal layer sizes, or, with
-    which="Ganupel" or "Burinex", that design beside Dofipel, or, with which="Rogizen", that design beside Ganupel
-    (random weights, bfloat16): decode throughput at batch 1, 8 and 64
+    which="Ganupel" or "Burinex", that design beside Dofipel, or, with which="Rogizen" or "Selinex", that design beside
+    Ganupel (random weights, bfloat16): decode throughput at batch 1, 8 and 64
     after 512-token prompts (captured steps, device time), prefill throughput of one 2,048-token prompt, and the
     per-kernel tables of both. Zemivik once without a mask (the attention work of Llama's) and once with a window
     of 1,024 tokens that keeps the first four. The shared vocabulary is kept small so that the layers, not the
@@ -549,7 +572,7 @@ def run_designs(args, pk: dict, which: str = "Zemivik") -> str:
     vocab = 32000
     shapes = [("1B layer sizes", CONFIG_1B), ("8B layer sizes", CONFIG_8B)]
     steps = min(args.steps, 64)
-    beside = {"Ganupel": "Dofipel", "Burinex": "Dofipel", "Rogizen": "Ganupel"}.get(which, "Llama")
+    beside = {"Ganupel": "Dofipel", "Burinex": "Dofipel", "Rogizen": "Ganupel", "Selinex": "Ganupel"}.get(which, "Llama")
     lines = [f"{which} beside {beside} at equal layer sizes, {n_layers} layers, vocabulary {vocab}, bfloat16, random weights "
              f"(peaks: {pk['hbm_gbs']:.0f} GB/s, {pk['bf16_tflops']:.0f} TFLOP/s, {pk['source']}).", "",
              "| layer sizes | design | decode b1 tok/s | ms/step | decode b8 tok/s | ms/step | decode b64 tok/s | ms/step | "
@@ -575,6 +598,9 @@ def run_designs(args, pk: dict, which: str = "Zemivik") -> str:
         if which == "Rogizen":
             designs = [("Ganupel, window 1024", ganupel_config(d, hq, hkv, hd, ff, vocab, n_layers, 1024)),
                        ("Rogizen, chunks of 1024", rogizen_config(d, hq, hkv, hd, ff, vocab, n_layers, 1024))]
+        if which == "Selinex":
+            designs = [("Ganupel, window 1024", ganupel_config(d, hq, hkv, hd, ff, vocab, n_layers, 1024)),
+                       ("Selinex, window 1024", selinex_config(d, hq, hkv, hd, ff, vocab, n_layers, 1024))]
         for design, cfg in designs:
             folder = scratch_folder("llmie_bench_design_")
             write_random_model(cfg, folder, seed=3, std=0.02)
@@ -696,8 +722,8 @@ def run_ours(args):
             with open(args.per_kernel_out, "w", encoding="utf-8") as f:
                 f.write(text + "\n")
         return 0
-    if args.designs or args.dofipel or args.ganupel or args.burinex or args.rogizen:
-        text = run_designs(args, pk, "Rogizen" if args.rogizen else "Burinex" if args.burinex else "Ganupel" if args.ganupel
+    if args.designs or args.dofipel or args.ganupel or args.burinex or args.rogizen or args.selinex:
+        text = run_designs(args, pk, "Selinex" if args.selinex else "Rogizen" if args.rogizen else "Burinex" if args.burinex else "Ganupel" if args.ganupel
                            else "Dofipel" if args.dofipel else "Zemivik")
         print(text)
         if args.per_kernel_out:
@@ -883,6 +909,10 @@ def main():
     ap.add_argument("--rogizen", action="store_true",
                     help="the same comparison for Rogizen (attention in chunks behind a short convolution, state space "
                          "layers, the embedding mixed into the stream) beside Ganupel, the closest design")
+    ap.add_argument("--selinex", action="store_true",
+                    help="the same comparison for Selinex (norms in front of and behind every branch; window attention "
+                         "beside gated linear attention or time mixing, gated delta rule layers, a router over groups of "
+                         "experts) beside Ganupel, the closest design")
     ap.add_argument("--heads", type=int, default=32, help="query heads of --attention-sweep")
     ap.add_argument("--kv-heads", type=int, default=8, help="KV heads of --attention-sweep")
     ap.add_argument("--head-dim", type=int, default=64, choices=[64, 128], help="head size of --attention-sweep")

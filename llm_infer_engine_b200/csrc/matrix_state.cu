@@ -184,8 +184,12 @@ struct StateArgs {
   float* o;                 // float32 [T, H * Dv]
   int q_ld, k_ld, v_ld, H, G, D, Dv, vec;
   float q_scale;
+  float* ws;                // long pieces in chunks side by side: [n_seqs, n_chunks, H, D, Dv], else null
+  float* prod;              // ... and the products of the chunks' decays, [n_seqs, n_chunks, H, D]
+  int chunk, n_chunks;      // tokens a chunk (a multiple of the tile), chunks of the longest piece (1: whole pieces)
 };
 
+// Four adjacent elements as float32; entries from `left` on are zeros. `vec`: one aligned access.
 template <typename T>
 __device__ __forceinline__ float4 load_row4(const T* p, int left, bool vec) {
   if (vec) {
@@ -200,31 +204,99 @@ __device__ __forceinline__ float4 load_row4(const T* p, int left, bool vec) {
                      left > 3 ? to_f32(p[3]) : 0.f);
 }
 
-constexpr int kScanTile = 8;           // tokens staged at a time
-constexpr int kScanBlock = 128;
+// Asks for four adjacent elements into shared memory, behind this thread's next commit; entries from `left` on become
+// zeros. Without `vec` (one aligned access) they are loaded and stored here and now.
+template <typename T>
+__device__ __forceinline__ void stage_row4(T* dst, const T* src, int left, bool vec) {
+  if (vec) {
+    const unsigned d = (unsigned)__cvta_generic_to_shared(dst);
+    const int n = left > 0 ? (int)(4 * sizeof(T)) : 0;
+    if (sizeof(T) == 4) asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(n) : "memory");
+    else asm volatile("cp.async.ca.shared.global [%0], [%1], 8, %2;" ::"r"(d), "l"(src), "r"(n) : "memory");
+    return;
+  }
+#pragma unroll
+  for (int e = 0; e < 4; ++e) dst[e] = e < left ? src[e] : from_f32<T>(0.f);
+}
 
-// grid (column tiles, heads, sequences). A column of the state is S lanes' work (S = 8, 16 or 32); lane s of them keeps the
-// rows 4 (s + S i) + e, i < R / 4, e < 4, in registers over the whole piece. Tiles of kScanTile tokens' decays, keys,
-// queries and values go through shared memory (two buffers); the next tile's are on their way in registers while a tile is
-// worked on. What the eight tokens of a tile read from the state is reduced over the lanes together: a step halves the
-// number of values and of lanes, so eight sums cost seven exchanges.
-template <typename TQ, typename TV, int FORM, int R, int S>
-__global__ void __launch_bounds__(kScanBlock) channel_scan_kernel(const StateArgs a) {
-  constexpr int DP = R * S;                                     // rows, padded
-  constexpr int COLS = kScanBlock / S;
-  constexpr int NARR = FORM == kFormDelta ? 2 : 3;              // q, k (, decays)
-  constexpr int RUNS = kScanTile * DP / 4;                      // runs of four in one staged array
-  constexpr int NV = (RUNS + kScanBlock - 1) / kScanBlock;
-  constexpr int CG = 32 / S;                                    // columns a warp
-  constexpr int BUF = kScanTile * (NARR * DP + COLS + 4);
-  extern __shared__ __align__(16) float scan_smem[];
+constexpr int kScanTile = 8;           // tokens staged at a time
+
+// Pairs of float32 in one register pair (two adjacent rows of a column): one instruction works on both.
+using pair_t = unsigned long long;
+__device__ __forceinline__ pair_t pair_of(float lo, float hi) {
+  pair_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ float2 pair_split(pair_t v) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+  return r;
+}
+__device__ __forceinline__ float pair_sum(pair_t v) { const float2 f = pair_split(v); return f.x + f.y; }
+__device__ __forceinline__ pair_t pair_fma(pair_t a, pair_t b, pair_t c) {
+  pair_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ pair_t pair_mul(pair_t a, pair_t b) {
+  pair_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+
+// The shape of a scan: a thread keeps C adjacent columns and R rows of them, S lanes share a column, NT threads a block.
+template <int C_, int R_, int S_, int NT_>
+struct ScanShape {
+  static constexpr int C = C_, R = R_, S = S_, NT = NT_;
+};
+
+// How a block of the scan lays out shared memory, in bytes: a ring of raw tiles, then two tiles in float32.
+template <typename TQ, typename TV, int FORM, typename SH>
+struct ScanLayout {
+  static constexpr int DP = SH::R * SH::S;                       // rows, padded
+  static constexpr int COLS = SH::NT / SH::S * SH::C;
+  static constexpr int NARR = FORM == kFormDelta ? 2 : 3;        // q, k (, decays)
+  static constexpr int RUNS = kScanTile * DP / 4;                // runs of four in one staged array
+  static constexpr int STAGES = DP > 256 ? 2 : 4;
+  static constexpr int RAW_Q = RUNS * 4 * (int)sizeof(TQ);
+  static constexpr int RAW_G = FORM == kFormDelta ? 0 : RUNS * 16;
+  static constexpr int RAW_V = kScanTile * COLS * (int)sizeof(TV);
+  static constexpr int RAW = 2 * RAW_Q + RAW_G + RAW_V + kScanTile * 16;
+  static constexpr int TILE = kScanTile * (NARR * DP + COLS + 4) * 4;
+  static constexpr size_t BYTES = (size_t)STAGES * RAW + 2 * TILE;
+};
+
+// grid (column tiles, heads, sequences). C adjacent columns of the state are S lanes' work; lane s of them keeps the rows
+// 4 (s + S i) + e, i < R / 4, e < 4, in registers over the whole piece, so that an entry of a key, query or decay that is
+// read from shared memory serves C columns. Tiles of kScanTile tokens' decays, keys, queries and values travel through a
+// ring of raw tiles (asynchronous copies, a few tiles ahead; every thread waits for, and converts, what it asked for
+// itself) into one of two float32 tiles, the next while the current one is worked on. Tokens behind the piece's end are
+// staged as ones that leave the state as it is. What the eight tokens of a tile read from the state is reduced over the
+// lanes together: a step halves the number of values and of lanes.
+//
+// Long pieces of forms 0 and 1, whose end state is linear in the start state: a piece is cut into chunks, grid z =
+// (sequence, chunk). OUT false runs every chunk but a sequence's last from a zero state, without outputs, and leaves its
+// end state in ws[c + 1] and the product of its decays in prod[c + 1]; a chain over the chunks makes ws[c] the state that
+// chunk c starts from; OUT true runs every chunk from there.
+template <typename TQ, typename TV, int FORM, typename SH, bool OUT>
+__global__ void __launch_bounds__(SH::NT) channel_scan_kernel(const StateArgs a) {
+  using L = ScanLayout<TQ, TV, FORM, SH>;
+  constexpr int C = SH::C, R = SH::R, S = SH::S, NT = SH::NT;
+  constexpr int DP = L::DP, COLS = L::COLS, RUNS = L::RUNS, STAGES = L::STAGES;
+  constexpr int NV = (RUNS + NT - 1) / NT;
+  constexpr int CG = 32 / S;                                    // groups of columns a warp
+  constexpr int VRUNS = kScanTile * COLS / 4;
+  constexpr int VV = (VRUNS + NT - 1) / NT;
+  constexpr int P = R / 2;                                      // pairs of rows a thread
+  extern __shared__ __align__(16) char scan_smem[];
   pdl_launch_dependents();
   const int tid = threadIdx.x;
-  const int s = tid & (S - 1), col = tid / S;
+  const int s = tid & (S - 1), col = tid / S * C;
   const int j0 = blockIdx.x * COLS, j = j0 + col;
-  const int h = blockIdx.y, seq = blockIdx.z, g = h / (a.H / a.G);
+  const int h = blockIdx.y, g = h / (a.H / a.G);
+  const int seq = blockIdx.z / a.n_chunks, chunk = blockIdx.z - seq * a.n_chunks;
   const int D = a.D, Dv = a.Dv;
-  const bool live = j < Dv;
   float4 bo[FORM == kFormBonus ? R / 4 : 1];
   if (FORM == kFormBonus) {
 #pragma unroll
@@ -234,72 +306,128 @@ __global__ void __launch_bounds__(kScanBlock) channel_scan_kernel(const StateArg
     }
   }
   pdl_wait();
-  const int t0 = a.cu_q[seq], t1 = a.cu_q[seq + 1];
+  const int seq_end = a.cu_q[seq + 1];
+  const int t0 = a.cu_q[seq] + chunk * a.chunk, t1 = a.n_chunks > 1 ? min(t0 + a.chunk, seq_end) : seq_end;
   if (t0 >= t1) return;
-  float* st = a.state + (((size_t)a.seq_slot[seq] * a.H + h) * D) * Dv + (live ? j : Dv - 1);
-  float4 St[R / 4];
-#pragma unroll
-  for (int i = 0; i < R / 4; ++i) {
-    const int row = 4 * (s + S * i);
-    St[i].x = row < D ? st[(size_t)row * Dv] : 0.f;
-    St[i].y = row + 1 < D ? st[(size_t)(row + 1) * Dv] : 0.f;
-    St[i].z = row + 2 < D ? st[(size_t)(row + 2) * Dv] : 0.f;
-    St[i].w = row + 3 < D ? st[(size_t)(row + 3) * Dv] : 0.f;
-  }
+  if (!OUT && t1 >= seq_end) return;                            // nobody needs the last chunk's end state
   const TQ* qb = reinterpret_cast<const TQ*>(a.q) + (size_t)g * D;
   const TQ* kb = reinterpret_cast<const TQ*>(a.k) + (size_t)g * D;
   const float* gb = FORM == kFormDelta ? nullptr : a.gate + (size_t)g * D;
   const TV* vb = reinterpret_cast<const TV*>(a.v) + (size_t)h * Dv;
   const size_t GD = (size_t)a.G * D;
-  float4 fq[NV], fk[NV], fg[FORM == kFormDelta ? 1 : NV];
-  float fv = 0.f, fs = 0.f;
-  constexpr int VN = kScanTile * COLS;                          // 32, 64 or 128 values: one a thread
-  auto fetch = [&](int t) {
+  auto raw_q = [&](int st) { return reinterpret_cast<TQ*>(scan_smem + st * L::RAW); };
+  auto raw_k = [&](int st) { return reinterpret_cast<TQ*>(scan_smem + st * L::RAW + L::RAW_Q); };
+  auto raw_g = [&](int st) { return reinterpret_cast<float*>(scan_smem + st * L::RAW + 2 * L::RAW_Q); };
+  auto raw_v = [&](int st) { return reinterpret_cast<TV*>(scan_smem + st * L::RAW + 2 * L::RAW_Q + L::RAW_G); };
+  auto raw_s = [&](int st) { return reinterpret_cast<float*>(scan_smem + st * L::RAW + 2 * L::RAW_Q + L::RAW_G + L::RAW_V); };
+  auto ask = [&](int t, int st) {                               // tile of tokens t .. into the ring's place st
+    if (t < t1) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int run = tid + i * NT;
+        if (run < RUNS) {
+          const int tt = run / (DP / 4), row = (run % (DP / 4)) * 4;
+          const int left = t + tt < t1 ? D - row : 0;
+          const size_t tok = t + tt < t1 ? t + tt : t1 - 1;
+          const int at = left > 0 ? row : 0;
+          stage_row4<TQ>(raw_q(st) + run * 4, qb + tok * a.q_ld + at, left, a.vec & 1);
+          stage_row4<TQ>(raw_k(st) + run * 4, kb + tok * a.k_ld + at, left, a.vec & 1);
+          if (FORM != kFormDelta) stage_row4<float>(raw_g(st) + run * 4, gb + tok * GD + at, left, a.vec & 1);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < VV; ++i) {
+        const int run = tid + i * NT;
+        if (run < VRUNS) {
+          const int tt = run / (COLS / 4), jj = j0 + (run % (COLS / 4)) * 4;
+          const int left = t + tt < t1 ? Dv - jj : 0;
+          const size_t tok = t + tt < t1 ? t + tt : t1 - 1;
+          stage_row4<TV>(raw_v(st) + run * 4, vb + tok * a.v_ld + (left > 0 ? jj : 0), left, a.vec & 2);
+        }
+      }
+      if (FORM == kFormDelta && tid < kScanTile && t + tid < t1) {
+        const size_t tok = t + tid;
+        const unsigned d = (unsigned)__cvta_generic_to_shared(raw_s(st) + tid * 4);
+        asm volatile("cp.async.ca.shared.global [%0], [%1], 8;" ::"r"(d), "l"(a.scal + (tok * a.H + h) * 2) : "memory");
+        asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(d + 8), "l"(a.qk + tok * a.G + g) : "memory");
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  float4 fq[NV], fk[NV], fg[FORM == kFormDelta ? 1 : NV], fv[VV], fs;
+  auto take = [&](int st) {                                     // this thread's part of a raw tile, as float32
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      const int run = tid + i * kScanBlock;
-      const int tt = run / (DP / 4), row = (run % (DP / 4)) * 4;
-      const int left = run < RUNS && t + tt < t1 ? D - row : 0;
-      const size_t tok = t + tt;
-      fq[i] = load_row4<TQ>(qb + tok * a.q_ld + row, left, a.vec);
-      fk[i] = load_row4<TQ>(kb + tok * a.k_ld + row, left, a.vec);
-      if (FORM != kFormDelta) fg[i] = load_row4<float>(gb + tok * GD + row, left, a.vec);
+      const int run = tid + i * NT;
+      if (run < RUNS) {
+        fq[i] = load_row4<TQ>(raw_q(st) + run * 4, 4, true);
+        fk[i] = load_row4<TQ>(raw_k(st) + run * 4, 4, true);
+        if (FORM != kFormDelta) fg[i] = load_row4<float>(raw_g(st) + run * 4, 4, true);
+      }
     }
-    if (tid < VN) {
-      const int tt = tid / COLS, jj = j0 + tid % COLS;
-      fv = t + tt < t1 && jj < Dv ? to_f32(vb[(size_t)(t + tt) * a.v_ld + jj]) : 0.f;
-    }
-    if (FORM == kFormDelta && tid < kScanTile * 4) {
-      const int tt = tid >> 2, e = tid & 3;
-      fs = 0.f;
-      if (t + tt < t1 && e < 2) fs = a.scal[((size_t)(t + tt) * a.H + h) * 2 + e];
-      if (t + tt < t1 && e == 2) fs = a.qk[(size_t)(t + tt) * a.G + g];
-    }
+#pragma unroll
+    for (int i = 0; i < VV; ++i)
+      if (tid + i * NT < VRUNS) fv[i] = load_row4<TV>(raw_v(st) + (tid + i * NT) * 4, 4, true);
+    if (FORM == kFormDelta && tid < kScanTile) fs = *reinterpret_cast<const float4*>(raw_s(st) + tid * 4);
   };
-  fetch(t0);
-  int buf = 0;
-  for (int t = t0; t < t1; t += kScanTile, buf ^= 1) {
-    float* base = scan_smem + buf * BUF;
-    float *sq = base, *sk = base + kScanTile * DP, *sg = base + 2 * kScanTile * DP, *sv = base + NARR * kScanTile * DP,
+  auto tile = [&](int buf) { return reinterpret_cast<float*>(scan_smem + STAGES * L::RAW + buf * L::TILE); };
+  auto put = [&](int t, int buf) {
+    float *sq = tile(buf), *sk = sq + kScanTile * DP, *sg = sk + kScanTile * DP, *sv = sq + L::NARR * kScanTile * DP,
           *sc = sv + kScanTile * COLS;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      const int run = tid + i * kScanBlock;
+      const int run = tid + i * NT;
       if (run < RUNS) {
         reinterpret_cast<float4*>(sq)[run] = make_float4(fq[i].x * a.q_scale, fq[i].y * a.q_scale, fq[i].z * a.q_scale,
                                                          fq[i].w * a.q_scale);
         reinterpret_cast<float4*>(sk)[run] = fk[i];
-        if (FORM != kFormDelta) reinterpret_cast<float4*>(sg)[run] = fg[i];
+        if (FORM != kFormDelta)
+          reinterpret_cast<float4*>(sg)[run] = t + run / (DP / 4) < t1 ? fg[i] : make_float4(1.f, 1.f, 1.f, 1.f);
       }
     }
-    if (tid < VN) sv[tid] = fv;
-    if (FORM == kFormDelta && tid < kScanTile * 4) sc[tid] = fs;
-    __syncthreads();
-    if (t + kScanTile < t1) fetch(t + kScanTile);
+#pragma unroll
+    for (int i = 0; i < VV; ++i)
+      if (tid + i * NT < VRUNS) reinterpret_cast<float4*>(sv)[tid + i * NT] = fv[i];
+    if (FORM == kFormDelta && tid < kScanTile)
+      reinterpret_cast<float4*>(sc)[tid] = t + tid < t1 ? fs : make_float4(0.f, 1.f, 0.f, 0.f);
+  };
+#pragma unroll
+  for (int i = 0; i < STAGES - 1; ++i) ask(t0 + i * kScanTile, i);
+  const size_t place = ((size_t)seq * a.n_chunks + chunk) * a.H + h;              // of (sequence, chunk, head)
+  float* st = a.state + (((size_t)a.seq_slot[seq] * a.H + h) * D) * Dv + j;
+  const float* start = OUT && a.n_chunks > 1 ? a.ws + place * D * Dv + j : st;
+  pair_t St[C][P];                                              // pair p of column c: rows row_of(p) and the next
+  auto row_of = [&](int p) { return 4 * (s + S * (p / 2)) + 2 * (p & 1); };
+#pragma unroll
+  for (int p = 0; p < P; ++p)
+#pragma unroll
+    for (int c = 0; c < C; ++c) {
+      const int row = row_of(p);
+      const bool ok = OUT && j + c < Dv;
+      St[c][p] = pair_of(ok && row < D ? start[(size_t)row * Dv + c] : 0.f,
+                         ok && row + 1 < D ? start[(size_t)(row + 1) * Dv + c] : 0.f);
+    }
+  pair_t decays[OUT ? 1 : P];                                   // the product of the chunk's decays
+#pragma unroll
+  for (int p = 0; p < (OUT ? 1 : P); ++p) decays[p] = pair_of(1.f, 1.f);
+  asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
+  take(0);
+  put(t0, 0);
+  __syncthreads();
+  int ring = 0, buf = 0;                                        // the current tile's places
+  for (int t = t0; t < t1; t += kScanTile, buf ^= 1) {
     const int n = min(kScanTile, t1 - t);
-    float acc[kScanTile];
-    float part[FORM == kFormBonus ? S / 4 : 1];                 // the bonus's share of q . k: a warp's columns take turns
-    if (FORM == kFormBonus) {
+    const bool more = t + kScanTile < t1;
+    // the place of the tile before the current one is free: this thread has converted its part of it
+    ask(t + (STAGES - 1) * kScanTile, (ring + STAGES - 1) % STAGES);
+    ring = (ring + 1) % STAGES;
+    asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
+    if (more) take(ring);
+    const float *sq = tile(buf), *sk = sq + kScanTile * DP, *sg = sk + kScanTile * DP,
+                *sv = sq + L::NARR * kScanTile * DP, *sc = sv + kScanTile * COLS;
+    float acc[kScanTile * C];                                   // token tt, column c at tt * C + c
+    float part[FORM == kFormBonus ? S / 4 : 1];                 // the bonus's share of q . k: a warp's groups take turns
+    if (FORM == kFormBonus && OUT) {
       const int cg = (tid & 31) / S;
 #pragma unroll
       for (int m = 0; m < S / 4; ++m) {
@@ -319,95 +447,165 @@ __global__ void __launch_bounds__(kScanBlock) channel_scan_kernel(const StateArg
     }
 #pragma unroll
     for (int tt = 0; tt < kScanTile; ++tt) {
-      acc[tt] = 0.f;
-      if (tt < n) {
-        const float v = sv[tt * COLS + col];
-        const float4* q4 = reinterpret_cast<const float4*>(sq + tt * DP) + s;
-        const float4* k4 = reinterpret_cast<const float4*>(sk + tt * DP) + s;
-        const float4* g4 = reinterpret_cast<const float4*>(sg + tt * DP) + s;
-        if (FORM == kFormDelta) {
-          float4 h4 = make_float4(0.f, 0.f, 0.f, 0.f), r4 = h4;
-          float4 kk[R / 4];
+      const ulonglong2* q2 = reinterpret_cast<const ulonglong2*>(sq + tt * DP) + s;
+      const ulonglong2* k2 = reinterpret_cast<const ulonglong2*>(sk + tt * DP) + s;
+      const ulonglong2* g2 = reinterpret_cast<const ulonglong2*>(sg + tt * DP) + s;
+      float v[C];
+      if constexpr (C == 4) {
+        const float4 f = *reinterpret_cast<const float4*>(sv + tt * COLS + col);
+        v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+      } else {
+        const float2 f = *reinterpret_cast<const float2*>(sv + tt * COLS + col);
+        v[0] = f.x; v[1] = f.y;
+      }
+      if constexpr (FORM == kFormDelta) {
+        pair_t held[C], read[C], kk[P];
 #pragma unroll
-          for (int i = 0; i < R / 4; ++i) {
-            kk[i] = k4[S * i];
-            const float4 q = q4[S * i];
-            h4.x = fmaf(kk[i].x, St[i].x, h4.x);
-            h4.y = fmaf(kk[i].y, St[i].y, h4.y);
-            h4.z = fmaf(kk[i].z, St[i].z, h4.z);
-            h4.w = fmaf(kk[i].w, St[i].w, h4.w);
-            r4.x = fmaf(q.x, St[i].x, r4.x);
-            r4.y = fmaf(q.y, St[i].y, r4.y);
-            r4.z = fmaf(q.z, St[i].z, r4.z);
-            r4.w = fmaf(q.w, St[i].w, r4.w);
+        for (int c = 0; c < C; ++c) held[c] = read[c] = 0ull;
+#pragma unroll
+        for (int i = 0; i < R / 4; ++i) {
+          const ulonglong2 k = k2[S * i], q = q2[S * i];
+          kk[2 * i] = k.x;
+          kk[2 * i + 1] = k.y;
+#pragma unroll
+          for (int c = 0; c < C; ++c) {
+            held[c] = pair_fma(k.x, St[c][2 * i], held[c]);
+            held[c] = pair_fma(k.y, St[c][2 * i + 1], held[c]);
+            read[c] = pair_fma(q.x, St[c][2 * i], read[c]);
+            read[c] = pair_fma(q.y, St[c][2 * i + 1], read[c]);
           }
-          float held = (h4.x + h4.y) + (h4.z + h4.w);
+        }
+        const float4 scal = reinterpret_cast<const float4*>(sc)[tt];            // beta, g, q . k
+        const pair_t g = pair_of(scal.y, scal.y);
+        float h1[C];
 #pragma unroll
-          for (int off = 1; off < S; off <<= 1) held += __shfl_xor_sync(0xffffffffu, held, off);
-          const float beta = sc[tt * 4], gt = sc[tt * 4 + 1], qk = sc[tt * 4 + 2];
-          const float u = beta * (v - gt * held);
-          acc[tt] = gt * ((r4.x + r4.y) + (r4.z + r4.w)) + (s == 0 ? u * qk : 0.f);
+        for (int c = 0; c < C; ++c) h1[c] = pair_sum(held[c]);
 #pragma unroll
-          for (int i = 0; i < R / 4; ++i) {
-            St[i].x = fmaf(gt, St[i].x, kk[i].x * u);
-            St[i].y = fmaf(gt, St[i].y, kk[i].y * u);
-            St[i].z = fmaf(gt, St[i].z, kk[i].z * u);
-            St[i].w = fmaf(gt, St[i].w, kk[i].w * u);
+        for (int off = 1; off < S; off <<= 1)
+#pragma unroll
+          for (int c = 0; c < C; ++c) h1[c] += __shfl_xor_sync(0xffffffffu, h1[c], off);
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+          const float u = scal.x * (v[c] - scal.y * h1[c]);
+          acc[tt * C + c] = scal.y * pair_sum(read[c]) + (s == 0 ? u * scal.z : 0.f);
+          const pair_t uu = pair_of(u, u);
+#pragma unroll
+          for (int p = 0; p < P; ++p) St[c][p] = pair_fma(g, St[c][p], pair_mul(kk[p], uu));
+        }
+      } else {
+        pair_t r[C], vv[C];
+        float bonus = 0.f;
+        if (FORM == kFormBonus && OUT)
+          bonus = CG == 1 ? part[tt] : __shfl_sync(0xffffffffu, part[tt / CG], (tt % CG) * S + s);
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+          r[c] = FORM == kFormBonus ? pair_of(bonus * v[c], 0.f) : 0ull;
+          vv[c] = pair_of(v[c], v[c]);
+        }
+#pragma unroll
+        for (int i = 0; i < R / 4; ++i) {
+          ulonglong2 q;
+          if (OUT) q = q2[S * i];
+          const ulonglong2 k = k2[S * i], f = g2[S * i];
+          if (!OUT) {
+            decays[2 * i % (OUT ? 1 : P)] = pair_mul(decays[2 * i % (OUT ? 1 : P)], f.x);
+            decays[(2 * i + 1) % (OUT ? 1 : P)] = pair_mul(decays[(2 * i + 1) % (OUT ? 1 : P)], f.y);
           }
+#pragma unroll
+          for (int c = 0; c < C; ++c) {
+            pair_t &lo = St[c][2 * i], &hi = St[c][2 * i + 1];
+            if (FORM == kFormBonus && OUT) r[c] = pair_fma(q.y, hi, pair_fma(q.x, lo, r[c]));
+            lo = pair_fma(f.x, lo, pair_mul(k.x, vv[c]));
+            hi = pair_fma(f.y, hi, pair_mul(k.y, vv[c]));
+            if (FORM == kFormKeyDecay && OUT) r[c] = pair_fma(q.y, hi, pair_fma(q.x, lo, r[c]));
+          }
+        }
+#pragma unroll
+        for (int c = 0; c < C; ++c) acc[tt * C + c] = pair_sum(r[c]);
+      }
+    }
+    if constexpr (OUT) {
+      // 8 C sums over the group's S lanes: step b hands over the half of the values that bit b of the lane does not name
+      constexpr int VALUES = kScanTile * C;
+      int first = 0;                                              // which of the values this lane ends with
+#pragma unroll
+      for (int b = 0; (1 << b) < S; ++b) {
+        const int left = VALUES >> (b + 1);
+        if (left > 0) {
+          const bool up = (s >> b) & 1;
+#pragma unroll
+          for (int i = 0; i < VALUES / 2; ++i)
+            if (i < left)
+              acc[i] = (up ? acc[i + left] : acc[i]) + __shfl_xor_sync(0xffffffffu, up ? acc[i] : acc[i + left], 1 << b);
+          first += up ? left : 0;
         } else {
-          float r0 = 0.f, r1 = 0.f;
-          if (FORM == kFormBonus)
-            r0 = v * __shfl_sync(0xffffffffu, part[tt / CG], (tt % CG) * S + s);
+          acc[0] += __shfl_xor_sync(0xffffffffu, acc[0], 1 << b);
+        }
+      }
+      constexpr int KEPT = VALUES >= S ? VALUES / S : 1;
+      if (s < VALUES) {
 #pragma unroll
-          for (int i = 0; i < R / 4; ++i) {
-            const float4 q = q4[S * i], k = k4[S * i], f = g4[S * i];
-            if (FORM == kFormBonus) {
-              r0 = fmaf(q.x, St[i].x, r0);
-              r1 = fmaf(q.y, St[i].y, r1);
-              r0 = fmaf(q.z, St[i].z, r0);
-              r1 = fmaf(q.w, St[i].w, r1);
-            }
-            St[i].x = fmaf(f.x, St[i].x, k.x * v);
-            St[i].y = fmaf(f.y, St[i].y, k.y * v);
-            St[i].z = fmaf(f.z, St[i].z, k.z * v);
-            St[i].w = fmaf(f.w, St[i].w, k.w * v);
-            if (FORM == kFormKeyDecay) {
-              r0 = fmaf(q.x, St[i].x, r0);
-              r1 = fmaf(q.y, St[i].y, r1);
-              r0 = fmaf(q.z, St[i].z, r0);
-              r1 = fmaf(q.w, St[i].w, r1);
-            }
-          }
-          acc[tt] = r0 + r1;
+        for (int i = 0; i < KEPT; ++i) {
+          const int tt = (first + i) / C, c = (first + i) % C;
+          if (tt < n && j + c < Dv) a.o[(size_t)(t + tt) * a.H * Dv + (size_t)h * Dv + j + c] = acc[i];
         }
       }
     }
-    // eight sums over the column's lanes: lane s ends with token s & 7
-    float r4[4], r2[2];
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const bool up = s & 4;
-      r4[i] = (up ? acc[i + 4] : acc[i]) + __shfl_xor_sync(0xffffffffu, up ? acc[i] : acc[i + 4], 4);
-    }
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const bool up = s & 2;
-      r2[i] = (up ? r4[i + 2] : r4[i]) + __shfl_xor_sync(0xffffffffu, up ? r4[i] : r4[i + 2], 2);
-    }
-    const bool up = s & 1;
-    float r = (up ? r2[1] : r2[0]) + __shfl_xor_sync(0xffffffffu, up ? r2[0] : r2[1], 1);
-#pragma unroll
-    for (int off = 8; off < S; off <<= 1) r += __shfl_xor_sync(0xffffffffu, r, off);
-    if (live && s < n && s < 8) a.o[(size_t)(t + s) * a.H * Dv + (size_t)h * Dv + j] = r;
+    if (more) put(t + kScanTile, buf ^ 1);
+    __syncthreads();
   }
-  if (!live) return;
+  if (OUT && t1 < seq_end) return;                              // the slot's state is the last chunk's to write
+  float* end = OUT ? st : a.ws + (place + a.H) * D * Dv + j;
 #pragma unroll
-  for (int i = 0; i < R / 4; ++i) {
-    const int row = 4 * (s + S * i);
-    if (row < D) st[(size_t)row * Dv] = St[i].x;
-    if (row + 1 < D) st[(size_t)(row + 1) * Dv] = St[i].y;
-    if (row + 2 < D) st[(size_t)(row + 2) * Dv] = St[i].z;
-    if (row + 3 < D) st[(size_t)(row + 3) * Dv] = St[i].w;
+  for (int p = 0; p < P; ++p)
+#pragma unroll
+    for (int c = 0; c < C; ++c) {
+      const int row = row_of(p);
+      const float2 f = pair_split(St[c][p]);
+      if (j + c < Dv && row < D) end[(size_t)row * Dv + c] = f.x;
+      if (j + c < Dv && row + 1 < D) end[(size_t)(row + 1) * Dv + c] = f.y;
+    }
+  if (!OUT && blockIdx.x == 0 && col == 0) {
+#pragma unroll
+    for (int p = 0; p < (OUT ? 1 : P); ++p) {
+      const int row = row_of(p);
+      const float2 f = pair_split(decays[p]);
+      if (row < D) a.prod[(place + a.H) * D + row] = f.x;
+      if (row + 1 < D) a.prod[(place + a.H) * D + row + 1] = f.y;
+    }
+  }
+}
+
+// The chain over a sequence's chunks, a thread per element of the state: ws[0] = the slot's state, ws[c] = prod[c] (.)
+// ws[c - 1] + ws[c], so that ws[c] is where chunk c starts.
+__global__ void channel_chain_kernel(const StateArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int seq = blockIdx.y;
+  const size_t n_state = (size_t)a.H * a.D * a.Dv, n_rows = (size_t)a.H * a.D;
+  const size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (e >= n_state) return;
+  const int nc = (a.cu_q[seq + 1] - a.cu_q[seq] + a.chunk - 1) / a.chunk;
+  if (nc <= 0) return;
+  float S = a.state[(size_t)a.seq_slot[seq] * n_state + e];
+  float* w = a.ws + (size_t)seq * a.n_chunks * n_state + e;
+  const float* d = a.prod + (size_t)seq * a.n_chunks * n_rows + e / a.Dv;
+  w[0] = S;
+  constexpr int U = 4;                                          // loads of the next chunks ahead of the chain
+  for (int c0 = 1; c0 < nc; c0 += U) {
+    float x[U], f[U];
+#pragma unroll
+    for (int i = 0; i < U; ++i)
+      if (c0 + i < nc) {
+        x[i] = w[(size_t)(c0 + i) * n_state];
+        f[i] = d[(size_t)(c0 + i) * n_rows];
+      }
+#pragma unroll
+    for (int i = 0; i < U; ++i)
+      if (c0 + i < nc) {
+        S = fmaf(f[i], S, x[i]);
+        w[(size_t)(c0 + i) * n_state] = S;
+      }
   }
 }
 
@@ -571,9 +769,7 @@ __global__ void __launch_bounds__(512) state_step_kernel(const StateArgs a, cons
   for (int j = tid; j < Dv; j += NT)
     yr[j] = from_f32<TP>(part[j] * rn * p.norm_w[(size_t)h * p.norm_stride + j] * siluf_(to_f32(zr[j])));
   if (FORM != kFormDelta || !works) return;
-  float u[V];
-#pragma unroll
-  for (int e = 0; e < V; ++e) u[e] = su[c + e];
+  const float* u = su + c;
   const bool kept = D <= kStepRows * RG;                        // every row is still in registers
   for (int base = rg; base < D; base += kStepRows * RG) {
 #pragma unroll
@@ -665,27 +861,55 @@ extern "C" int llmie_shift_mix(const void* x, float* prev, const float* mu, cons
   return LLMIE_OK;
 }
 
-template <typename TQ, typename TV, int FORM, int R, int S>
+template <typename TQ, typename TV, int FORM, typename SH>
 static int channel_scan_launch(const StateArgs& a, int n_seqs, cudaStream_t stream) {
-  constexpr int NARR = FORM == kFormDelta ? 2 : 3;
-  constexpr size_t smem = 2 * sizeof(float) * kScanTile * (NARR * R * S + kScanBlock / S + 4);
-  auto kernel = channel_scan_kernel<TQ, TV, FORM, R, S>;
-  if (smem > 48 * 1024) {
-    const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  using L = ScanLayout<TQ, TV, FORM, SH>;
+  auto kernel = channel_scan_kernel<TQ, TV, FORM, SH, true>;
+  const dim3 grid((a.Dv + L::COLS - 1) / L::COLS, a.H, n_seqs * a.n_chunks), block(SH::NT);
+  if (L::BYTES > 48 * 1024) {
+    const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)L::BYTES);
     if (e != cudaSuccess) return (int)e;
   }
-  const int cols = kScanBlock / S;
-  launch_k(kernel, dim3((a.Dv + cols - 1) / cols, a.H, n_seqs), dim3(kScanBlock), smem, stream, a);
+  if constexpr (FORM != kFormDelta) {
+    if (a.n_chunks > 1) {
+      auto first = channel_scan_kernel<TQ, TV, FORM, SH, false>;
+      if (L::BYTES > 48 * 1024) {
+        const cudaError_t e = cudaFuncSetAttribute(first, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)L::BYTES);
+        if (e != cudaSuccess) return (int)e;
+      }
+      launch_k(first, grid, block, L::BYTES, stream, a);
+      const size_t n_state = (size_t)a.H * a.D * a.Dv;
+      launch_k(channel_chain_kernel, dim3((unsigned)((n_state + 255) / 256), n_seqs), dim3(256), 0, stream, a);
+    }
+  }
+  launch_k(kernel, grid, block, L::BYTES, stream, a);
   return LLMIE_OK;
 }
 
+// Four columns a thread where tokens do not wait for one another. The delta rule does: every token's write needs a sum over
+// the rows first, so fewer lanes share a column there, unless the step has too few warps to hide that sum behind one another
+// (which lanes add what then depends on how many sequences a step has; a float32 engine always takes the first way).
 template <typename TQ, typename TV, int FORM>
 static int channel_scan_sizes(const StateArgs& a, int n_seqs, cudaStream_t stream) {
-  if (a.D <= 32) return channel_scan_launch<TQ, TV, FORM, 4, 8>(a, n_seqs, stream);
-  if (a.D <= 64) return channel_scan_launch<TQ, TV, FORM, 8, 8>(a, n_seqs, stream);
-  if (a.D <= 128) return channel_scan_launch<TQ, TV, FORM, 16, 8>(a, n_seqs, stream);
-  if (a.D <= 256) return channel_scan_launch<TQ, TV, FORM, 16, 16>(a, n_seqs, stream);
-  return channel_scan_launch<TQ, TV, FORM, 16, 32>(a, n_seqs, stream);
+  if constexpr (FORM == kFormDelta) {
+    if (a.D <= 32) return channel_scan_launch<TQ, TV, FORM, ScanShape<2, 8, 4, 32>>(a, n_seqs, stream);
+    if constexpr (sizeof(TV) == 2) {
+      const long long warps = (long long)n_seqs * a.H * ((a.Dv + 31) / 32) * (a.D <= 64 ? 2 : 4);
+      if (a.D <= 64 && warps < 900) return channel_scan_launch<TQ, TV, FORM, ScanShape<2, 8, 8, 128>>(a, n_seqs, stream);
+      if (a.D > 64 && a.D <= 128 && warps < 900)
+        return channel_scan_launch<TQ, TV, FORM, ScanShape<2, 8, 16, 256>>(a, n_seqs, stream);
+    }
+    if (a.D <= 64) return channel_scan_launch<TQ, TV, FORM, ScanShape<2, 16, 4, 64>>(a, n_seqs, stream);
+    if (a.D <= 128) return channel_scan_launch<TQ, TV, FORM, ScanShape<2, 16, 8, 128>>(a, n_seqs, stream);
+    if (a.D <= 256) return channel_scan_launch<TQ, TV, FORM, ScanShape<2, 16, 16, 128>>(a, n_seqs, stream);
+    return channel_scan_launch<TQ, TV, FORM, ScanShape<2, 16, 32, 128>>(a, n_seqs, stream);
+  } else {
+    if (a.D <= 32) return channel_scan_launch<TQ, TV, FORM, ScanShape<4, 4, 8, 32>>(a, n_seqs, stream);
+    if (a.D <= 64) return channel_scan_launch<TQ, TV, FORM, ScanShape<4, 4, 16, 64>>(a, n_seqs, stream);
+    if (a.D <= 128) return channel_scan_launch<TQ, TV, FORM, ScanShape<4, 4, 32, 128>>(a, n_seqs, stream);
+    if (a.D <= 256) return channel_scan_launch<TQ, TV, FORM, ScanShape<4, 8, 32, 128>>(a, n_seqs, stream);
+    return channel_scan_launch<TQ, TV, FORM, ScanShape<4, 16, 32, 128>>(a, n_seqs, stream);
+  }
 }
 
 static inline bool aligned_rows(const void* p, int ld, int dt) {
@@ -694,22 +918,29 @@ static inline bool aligned_rows(const void* p, int ld, int dt) {
 
 // q, k (rows q_ld, k_ld apart) of q_dtype, v (v_ld apart) of v_dtype; form 0 and 1: gate float32 [T, G D] (form 1 also
 // bonus float32 [G D]); form 2: scal, qk as delta_prepare leaves them. state float32 [slots, H, D, Dv] is read and written;
-// o float32 [T, H Dv]. D up to 512.
+// o float32 [T, H Dv]. D up to 512. ws null: whole pieces (the only way for form 2); otherwise chunks of `chunk` tokens side
+// by side, n_chunks >= ceil(longest piece / chunk), ws float32 [n_seqs, n_chunks, H, D, Dv] and prod float32
+// [n_seqs, n_chunks, H, D] scratch.
 extern "C" int llmie_channel_scan(const void* q, int q_ld, const void* k, int k_ld, int q_dtype, float q_scale,
                                   const void* v, int v_ld, int v_dtype, const float* gate, const float* bonus,
                                   const float* scal, const float* qk, float* state, const int* cu_q, const int* seq_slot,
-                                  float* o, int n_seqs, int H, int G, int D, int Dv, int form, cudaStream_t stream) {
+                                  float* o, float* ws, float* prod, int chunk, int n_chunks, int n_seqs, int H, int G, int D,
+                                  int Dv, int form, cudaStream_t stream) {
   if (!q || !k || !v || !state || !o || n_seqs < 0 || H <= 0 || G <= 0 || H % G || D <= 0 || Dv <= 0 || q_ld < G * D ||
       k_ld < G * D || v_ld < H * Dv || form < 0 || form > 2)
     return LLMIE_ERR_BAD_ARG;
   if ((form != 2 && !gate) || (form == 1 && !bonus) || (form == 2 && (!scal || !qk))) return LLMIE_ERR_BAD_ARG;
   if (!dtype_ok(q_dtype) || !dtype_ok(v_dtype)) return LLMIE_ERR_DTYPE;
-  if (D > 512 || H > 65535 || n_seqs > 65535) return LLMIE_ERR_UNSUPPORTED_SIZE;
+  if (ws && (form == 2 || !prod || chunk <= 0 || chunk % kScanTile || n_chunks <= 0)) return LLMIE_ERR_BAD_ARG;
+  if (!ws) { chunk = 0; n_chunks = 1; }
+  if (D > 512 || H > 65535 || (long long)n_seqs * n_chunks > 65535) return LLMIE_ERR_UNSUPPORTED_SIZE;
   if (n_seqs == 0) return LLMIE_OK;
   const bool vec = D % 4 == 0 && aligned_rows(q, q_ld, q_dtype) && aligned_rows(k, k_ld, q_dtype) &&
                    (form == 2 || aligned_rows(gate, G * D, LLMIE_F32));
-  const StateArgs a{q, k, v, gate, bonus, scal, qk, state, cu_q, seq_slot, o, q_ld, k_ld, v_ld, H, G, D, Dv, vec ? 1 : 0,
-                    q_scale};
+  const bool vec_v = Dv % 4 == 0 && aligned_rows(v, v_ld, v_dtype);
+  const StateArgs a{q, k, v, gate, bonus, scal, qk, state, cu_q, seq_slot, o, q_ld, k_ld, v_ld, H, G, D, Dv,
+                    (vec ? 1 : 0) | (vec_v ? 2 : 0), q_scale, ws, prod, chunk, n_chunks};
+  if (form == 2 && (reinterpret_cast<uintptr_t>(scal) & 7u)) return LLMIE_ERR_ALIGNMENT;
   int rc = LLMIE_ERR_DTYPE;
 #define LLMIE_SCAN_FORM(TQ, TV)                                                \
   rc = form == 0   ? channel_scan_sizes<TQ, TV, kFormKeyDecay>(a, n_seqs, stream) \
@@ -779,7 +1010,7 @@ extern "C" int llmie_state_step(const void* q, int q_ld, const void* k, int k_ld
   const size_t smem = step_smem(D, Dv, V, nt);
   if (smem > 48 * 1024) return LLMIE_ERR_UNSUPPORTED_SIZE;
   const StateArgs a{q, k, v, nullptr, bonus, nullptr, nullptr, state, cu_q, seq_slot, nullptr, q_ld, k_ld, v_ld, H, G, D,
-                    Dv, 0, q_scale};
+                    Dv, 0, q_scale, nullptr, nullptr, 0, 1};
   const StepArgs p{x, Bt, gate_bias, ba, A, dt_bias, norm_w, z, out, x_ld, x_dtype, R, mode, ba_ld, b_off, a_off,
                    norm_stride, z_ld, inv_tau, unit_eps, norm_eps};
   const dim3 grid(H, n_seqs), block(nt);

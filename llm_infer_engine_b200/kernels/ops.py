@@ -2057,6 +2057,8 @@ def unit_scan(gates, proj, y_off: int, x_off: int, y_bias, x_bias, act: int, sta
 FORM_KEY_DECAY, FORM_BONUS, FORM_DELTA = 0, 1, 2      # csrc/matrix_state.cu
 GATE_POWER, GATE_DOUBLE_EXP = 0, 1                     # sigmoid(z)^(1/tau); exp(-exp(z)) with tanh in front of the product
 MAX_CHANNEL_DIM, MAX_GATE_RANK = 512, 512
+CHANNEL_CHUNK = 128           # tokens a chunk of a long piece
+CHANNEL_FULL_WARPS = 1024     # warps from which whole pieces are as fast as chunks
 
 
 def low_rank_gate(x, Bt, bias, out, mode: int, tau: float = 1.0):
@@ -2117,8 +2119,11 @@ def shift_mix(x, prev, mu, cu_q, tok_seq, seq_slot, out, single: bool = False):
 
 
 def channel_scan(form: int, q, k, v, state, cu_q, seq_slot, out, n_seqs: int, heads: int, groups: int, dim: int, vdim: int,
-                 q_scale: float = 1.0, gate=None, bonus=None, scal=None, qk=None):
-    """The recurrences of csrc/matrix_state.cu over pieces of any length. q, k [T, groups dim] of one type and v
+                 q_scale: float = 1.0, gate=None, bonus=None, scal=None, qk=None, max_len: Optional[int] = None):
+    """The recurrences of csrc/matrix_state.cu over pieces of any length. `max_len`: a bound on the longest piece; with it,
+    FORM_KEY_DECAY and FORM_BONUS run pieces of more than CHANNEL_CHUNK tokens in chunks side by side: always in
+    float32, so that a sequence's arithmetic does not depend on what else is in the step, and in bfloat16 where whole
+    pieces would leave the GPU short of warps. q, k [T, groups dim] of one type and v
     [T, heads vdim] (column slices allowed); state float32 [slots, heads, dim, vdim] is read and written; out float32
     [T, heads vdim]. FORM_KEY_DECAY, FORM_BONUS: gate float32 [T, groups dim] (and bonus float32 [groups dim]);
     FORM_DELTA: scal, qk of `delta_prepare`."""
@@ -2133,14 +2138,25 @@ def channel_scan(form: int, q, k, v, state, cu_q, seq_slot, out, n_seqs: int, he
                            ("scal", scal, (T, heads, 2)), ("qk", qk, (T, groups))):
         if t is not None:
             _need(t, name, torch.float32, shape)
+    ws = prod = None
+    chunk, n_chunks = CHANNEL_CHUNK, 1
+    short = v.dtype == torch.float32 or n_seqs * heads * -(-vdim // 16) * -(-min(dim, 128) // 32) < CHANNEL_FULL_WARPS
+    if form != FORM_DELTA and max_len is not None and max_len > chunk and short:
+        while n_seqs * -(-max_len // chunk) * heads * dim * vdim * 4 > SCAN_SCRATCH_BYTES and chunk < max_len:
+            chunk *= 2
+        n_chunks = -(-max_len // chunk)
+        if 2 <= n_chunks and n_seqs * n_chunks <= 65535:
+            ws = torch.empty((n_seqs, n_chunks, heads, dim, vdim), dtype=torch.float32, device=q.device)
+            prod = torch.empty((n_seqs, n_chunks, heads, dim), dtype=torch.float32, device=q.device)
     _work(2 * T * groups * dim * q.element_size() + T * heads * vdim * v.element_size() + _nbytes(gate, scal, qk, out) +
           8.0 * n_seqs * heads * dim * vdim, (8.0 if form == FORM_DELTA else 5.0) * T * heads * dim * vdim)
     f = _fn("matrix_state", "llmie_channel_scan",
-            [_c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_float, _c_void_p, _c_int, _c_int] + [_c_void_p] * 8 +
-            [_c_int] * 6 + [_c_void_p])
+            [_c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_float, _c_void_p, _c_int, _c_int] + [_c_void_p] * 10 +
+            [_c_int] * 8 + [_c_void_p])
     _check(f(q.data_ptr(), q_ld, k.data_ptr(), k_ld, _dt(q, "q"), float(q_scale), v.data_ptr(), v_ld, _dt(v, "v"),
              _ptr(gate), _ptr(bonus), _ptr(scal), _ptr(qk), state.data_ptr(), cu_q.data_ptr(), seq_slot.data_ptr(),
-             out.data_ptr(), n_seqs, heads, groups, dim, vdim, int(form), _stream()), "channel_scan")
+             out.data_ptr(), _ptr(ws), _ptr(prod), chunk, n_chunks, n_seqs, heads, groups, dim, vdim, int(form), _stream()),
+           "channel_scan")
     return out
 
 

@@ -147,7 +147,7 @@ class KeyDecayAttention(_MatrixState):
             ops.low_rank_gate(low, self.a2t, self.a2_bias, decay, ops.GATE_POWER, self.tau)
             read = torch.empty((T, nv), dtype=torch.float32, device=dev)
             ops.channel_scan(self.form, q, k, v, *self._state_args(ctx, unit), read, *self._geometry(ctx), q_scale=scale,
-                             gate=decay)
+                             gate=decay, max_len=ctx.max_q_len)
             ops.head_rmsnorm(read, self.norm_w, self.eps, out, self.v_dim, gate=z, gate_silu=True)
         trace.pop()
         trace.push("Output_proj")
@@ -232,7 +232,7 @@ class TimeMixing(_MatrixState):
             ops.low_rank_gate(low, self.w2t, self.w0, decay, ops.GATE_DOUBLE_EXP)
             read = torch.empty((T, nq), dtype=torch.float32, device=dev)
             ops.channel_scan(self.form, r, k, v, *self._state_args(ctx, unit), read, *self._geometry(ctx), gate=decay,
-                             bonus=self.bonus)
+                             bonus=self.bonus, max_len=ctx.max_q_len)
             ops.head_rmsnorm(read, self.norm_w, self.eps, out, self.dim, gate=z, gate_silu=True)
         trace.pop()
         trace.push("Output_proj")

@@ -907,8 +907,8 @@ static int channel_scan_sizes(const StateArgs& a, int n_seqs, cudaStream_t strea
     if (a.D <= 32) return channel_scan_launch<TQ, TV, FORM, ScanShape<4, 4, 8, 32>>(a, n_seqs, stream);
     if (a.D <= 64) return channel_scan_launch<TQ, TV, FORM, ScanShape<4, 4, 16, 64>>(a, n_seqs, stream);
     if (a.D <= 128) return channel_scan_launch<TQ, TV, FORM, ScanShape<4, 4, 32, 128>>(a, n_seqs, stream);
-    if (a.D <= 256) return channel_scan_launch<TQ, TV, FORM, ScanShape<4, 8, 32, 128>>(a, n_seqs, stream);
-    return channel_scan_launch<TQ, TV, FORM, ScanShape<4, 16, 32, 128>>(a, n_seqs, stream);
+    if (a.D <= 256) return channel_scan_launch<TQ, TV, FORM, ScanShape<2, 8, 32, 128>>(a, n_seqs, stream);
+    return channel_scan_launch<TQ, TV, FORM, ScanShape<2, 16, 32, 128>>(a, n_seqs, stream);
   }
 }
 

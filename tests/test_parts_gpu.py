@@ -28,7 +28,8 @@ def build(group, kind, params, dtype, tensors=None, seed=0, std=0.1):
     g = torch.Generator().manual_seed(seed)
     host = {}
     for name, ps in part.param_specs().items():
-        t = torch.rand(ps.shape, generator=g) + 0.5 if ps.role == "vector" else torch.randn(ps.shape, generator=g) * std
+        shape = tuple(abs(n) for n in ps.shape)                  # a negative entry: a size the checkpoint decides
+        t = torch.rand(shape, generator=g) + 0.5 if ps.role == "vector" else torch.randn(shape, generator=g) * std
         host[name] = t.to(torch.bfloat16).float()
     part.load({n: t.to(DEV, DTYPES[dtype]) for n, t in host.items()})
     return part, host

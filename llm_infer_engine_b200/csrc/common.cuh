@@ -108,10 +108,13 @@ struct GateForm {
   float alpha, limit;
 };
 constexpr int kActClamped = 5;
+// FAST: the approximate exponential and division, in front of a store that keeps 8 bits of the result.
+template <bool FAST = false>
 __device__ __forceinline__ float gated_pair(float g, float u, const GateForm& f) {
   if (f.act != kActClamped) return apply_act(g, f.act) * u;
   g = fminf(g, f.limit);
   u = fminf(fmaxf(u, -f.limit), f.limit);
+  if (FAST) return __fdividef(g, 1.f + __expf(fminf(-f.alpha * g, 80.f))) * (u + 1.f);
   return g / (1.f + expf(-f.alpha * g)) * (u + 1.f);
 }
 

@@ -90,7 +90,7 @@ __global__ void gated_act_kernel(const T* __restrict__ gate_up, T* __restrict__ 
     const int j = (int)(i - t * ff);
     const float g = to_f32(gate_up[t * 2 * ff + j]);
     const float u = to_f32(gate_up[t * 2 * ff + ff + j]);
-    out[i] = from_f32<T>(gated_pair(g, u, form));
+    out[i] = from_f32<T>(gated_pair<sizeof(T) == 2>(g, u, form));
   }
 }
 
@@ -106,7 +106,7 @@ __global__ void gated_act_vec_kernel(const T* __restrict__ gate_up, T* __restric
     load8(row + j, g);
     load8(row + ff + j, u);
 #pragma unroll
-    for (int e = 0; e < 8; ++e) o[e] = gated_pair(g[e], u[e], form);
+    for (int e = 0; e < 8; ++e) o[e] = gated_pair<sizeof(T) == 2>(g[e], u[e], form);
     store8(out + t * ff + j, o);
   }
 }

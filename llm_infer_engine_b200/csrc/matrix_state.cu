@@ -630,7 +630,7 @@ constexpr int kStepRows = 8;             // rows a thread keeps between the two 
 // grid (heads, sequences). A thread owns V adjacent columns (4 where the value size allows) and every RG-th row, RG the
 // block's threads over the columns' threads, so that a warp's accesses to the state are whole rows side by side.
 template <typename TQ, typename TP, int FORM, int V>
-__global__ void __launch_bounds__(512) state_step_kernel(const StateArgs a, const StepArgs p) {
+__global__ void __launch_bounds__(512, 2) state_step_kernel(const StateArgs a, const StepArgs p) {
   extern __shared__ __align__(16) float step_smem[];           // q [D] | k [D] | decays [D] | u [Dv] | partial sums
   __shared__ float red[32];
   pdl_launch_dependents();
